@@ -14,6 +14,7 @@ from . import sugizen  # registers Sugizen
 from . import tinuzen  # registers Tinuzen
 from . import vusalix  # registers Vusalix
 from . import bizepel  # registers Bizepel
+from . import bozavik  # registers Bozavik
 
 for _name in filter(None, (m.strip() for m in os.environ.get("ULTIMA_ARCH_MODULES", "").split(","))):
     importlib.import_module(_name)

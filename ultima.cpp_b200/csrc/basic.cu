@@ -16,7 +16,7 @@
 // ---------------------------------------------------------------------------------------
 template <typename TT>
 __global__ void embed_kernel(const TT* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ x, int width, int vocab, int* status) {
+                             float* __restrict__ x, int width, int vocab, int* status, float scale) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -25,13 +25,13 @@ __global__ void embed_kernel(const TT* __restrict__ table, const int* __restrict
     if (!ok && threadIdx.x == 0) atomicExch(status, 1);
     const TT* row = table + (long long)(ok ? id : 0) * width;
     for (int i = threadIdx.x; i < width; i += blockDim.x)
-        x[(long long)t * width + i] = ok ? to_f32<TT>(row[i]) : 0.f;
+        x[(long long)t * width + i] = ok ? to_f32<TT>(row[i]) * scale : 0.f;
 }
 
 // The same, eight values a thread and step: rows that begin on 16-byte boundaries.
 template <typename TT>
 __global__ void embed_vec_kernel(const TT* __restrict__ table, const int* __restrict__ ids,
-                                 float* __restrict__ x, int width, int vocab, int* status) {
+                                 float* __restrict__ x, int width, int vocab, int* status, float scale) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -43,29 +43,29 @@ __global__ void embed_vec_kernel(const TT* __restrict__ table, const int* __rest
         float v[8];
         load_vec<TT, 8>(row + i, v);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = ok ? v[j] : 0.f;
+        for (int j = 0; j < 8; ++j) v[j] = ok ? v[j] * scale : 0.f;
         store_vec<float, 8>(x + (long long)t * width + i, v);
     }
 }
 
 UB_API int ub_embed(const void* table, int table_dtype, const int* ids, float* x, int n_tokens,
-                    int width, int vocab, int* status, cudaStream_t st) {
+                    int width, int vocab, int* status, float scale, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     cudaError_t e;
     if (width % 8 == 0 && (((uintptr_t)table | (uintptr_t)x) & 15) == 0 && (table_dtype == UB_F32 || table_dtype == UB_BF16)) {
         int vt = 32;
         while (vt < 256 && vt * 16 < width) vt <<= 1;
         if (table_dtype == UB_F32)
-            e = ub_launch_dependent(embed_vec_kernel<float>, dim3(n_tokens), dim3(vt), 0, st, (const float*)table, ids, x, width, vocab, status);
+            e = ub_launch_dependent(embed_vec_kernel<float>, dim3(n_tokens), dim3(vt), 0, st, (const float*)table, ids, x, width, vocab, status, scale);
         else
-            e = ub_launch_dependent(embed_vec_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(vt), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status);
+            e = ub_launch_dependent(embed_vec_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(vt), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale);
         return (int)e;
     }
     const int threads = width >= 1024 ? 256 : 128;
     if (table_dtype == UB_F32)
-        e = ub_launch_dependent(embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, st, (const float*)table, ids, x, width, vocab, status);
+        e = ub_launch_dependent(embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, st, (const float*)table, ids, x, width, vocab, status, scale);
     else if (table_dtype == UB_BF16)
-        e = ub_launch_dependent(embed_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status);
+        e = ub_launch_dependent(embed_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale);
     else return UB_ERR_UNSUPPORTED;
     return (int)e;
 }
@@ -521,7 +521,7 @@ UB_API int ub_rmsnorm_add(float* y, const float* w, float* x, void* h, int h_dty
 // ---------------------------------------------------------------------------------------
 template <typename TI, typename TO>
 __global__ void glu_clamped_kernel(const TI* __restrict__ gu, TO* __restrict__ out, long long n, int F,
-                                   float limit, float alpha, float shift) {
+                                   float limit, float alpha, float shift, const float* __restrict__ row_gate, long long rg_stride) {
     pdl_trigger();
     pdl_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -531,16 +531,18 @@ __global__ void glu_clamped_kernel(const TI* __restrict__ gu, TO* __restrict__ o
     const float g = fminf(to_f32<TI>(gu[t * 2 * F + f]), limit);
     const float u = fminf(fmaxf(to_f32<TI>(gu[t * 2 * F + F + f]), -limit), limit);
     // an infinite alpha is the sigmoid's hard limit: the gate passes g where it is positive (a rectifier)
-    out[i] = from_f32<TO>((isinf(alpha) ? fmaxf(g, 0.f) : g / (1.0f + expf(-alpha * g))) * (u + shift));
+    float v = (isinf(alpha) ? fmaxf(g, 0.f) : g / (1.0f + expf(-alpha * g))) * (u + shift);
+    if (row_gate) v *= 1.0f / (1.0f + expf(-row_gate[t * rg_stride]));        // one sigmoid gate a row
+    out[i] = from_f32<TO>(v);
 }
 
 UB_API int ub_glu_clamped(const void* gu, int in_dtype, void* out, int out_dtype, int n_tokens, int F,
-                          float limit, float alpha, float shift, cudaStream_t st) {
+                          float limit, float alpha, float shift, const float* row_gate, long long rg_stride, cudaStream_t st) {
     const long long n = (long long)n_tokens * F;
     if (n <= 0) return 0;
     const unsigned grid = (unsigned)((n + 255) / 256);
     cudaError_t e;
-#define LAUNCH(TI, TO) e = ub_launch_dependent(glu_clamped_kernel<TI, TO>, dim3(grid), dim3(256), 0, st, (const TI*)gu, (TO*)out, n, F, limit, alpha, shift)
+#define LAUNCH(TI, TO) e = ub_launch_dependent(glu_clamped_kernel<TI, TO>, dim3(grid), dim3(256), 0, st, (const TI*)gu, (TO*)out, n, F, limit, alpha, shift, row_gate, rg_stride)
     if (in_dtype == UB_F32 && out_dtype == UB_F32) LAUNCH(float, float);
     else if (in_dtype == UB_F32 && out_dtype == UB_BF16) LAUNCH(float, __nv_bfloat16);
     else if (in_dtype == UB_BF16 && out_dtype == UB_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -24,6 +24,9 @@ struct SimtExtra {
     const int4* tiles;              // grouped: (matrix, first sorted row, rows, unused) for every block of rows
     const int* n_tiles;             // grouped: tiles in use (on the device)
     const int* src_rows;            // grouped, optional: the row of A behind a sorted row
+    // the gate product's constants: g' / (1 + exp(-alpha g')) * (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit);
+    // the defaults give silu(g) * u
+    float limit = INFINITY, alpha = 1.0f, shift = 0.0f;
 };
 
 template <typename TA, typename TW, typename TO, int EPI>
@@ -101,7 +104,10 @@ gemm_simt_kernel(const TA* __restrict__ A, const TW* __restrict__ W, const TW* _
             TO* p = out + (long long)m * ldo + n;
             if (EPI == EPI_STORE) *p = from_f32<TO>(acc[i][j]);
             else if (EPI == EPI_ADD) *p = from_f32<TO>(to_f32<TO>(*p) + acc[i][j]);
-            else { const float g = acc[i][j]; *p = from_f32<TO>(g / (1.0f + expf(-g)) * acc2[i][j]); }
+            else {
+                const float g = fminf(acc[i][j], ex.limit), u = fminf(fmaxf(acc2[i][j], -ex.limit), ex.limit);
+                *p = from_f32<TO>(g / (1.0f + expf(-ex.alpha * g)) * (u + ex.shift));
+            }
         }
     }
 }
@@ -155,12 +161,14 @@ UB_API int ub_gemm_simt_batched(const void* A, int a_dtype, const void* W, int w
 
 // Sorted rows against the matrix each tile names: out[sorted row, :] = A[src_rows[sorted row] or the row, :] W_e^T (with
 // EPI_SWIGLU the second matrix W2_e is the same distance from W2).  ``max_tiles``: the most tiles the launch can need.
+// ``gate`` (host, three floats or null): limit, alpha and shift of the gate product.
 UB_API int ub_gemm_simt_grouped(const void* A, int a_dtype, const void* W, const void* W2, int w_dtype, void* out, int o_dtype,
                                 int N, int K, long long lda, long long ldw, long long ldo, long long w_bs, const void* tiles,
-                                const int* n_tiles, const int* src_rows, int max_tiles, int epi, cudaStream_t st) {
+                                const int* n_tiles, const int* src_rows, int max_tiles, int epi, const float* gate, cudaStream_t st) {
     if (N <= 0 || max_tiles <= 0) return 0;
     if (!tiles || !n_tiles || epi == EPI_ADD) return UB_ERR_ARG;
     SimtExtra ex{0, w_bs, 0, (const int4*)tiles, n_tiles, src_rows};
+    if (gate) { ex.limit = gate[0]; ex.alpha = gate[1]; ex.shift = gate[2]; }
     return dispatch(A, a_dtype, W, W2, w_dtype, out, o_dtype, 0, N, K, lda, ldw, ldo, epi, st, ex, 1, max_tiles);
 }
 

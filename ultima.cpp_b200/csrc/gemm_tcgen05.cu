@@ -53,7 +53,14 @@ struct GemmParams {
     // EPI_STORE: what is stored is a function of the sum: 0 the sum itself, 1 the exact GELU 0.5 v (1 + erf(v / sqrt 2)),
     // 2 the squared rectifier max(v, 0)^2 (whole K only: a slice's partial sum has no activation)
     int unary;
+    // every stored result (not the adding epilogue's) times the sigmoid of mul[t * mul_ld + n * mul_col] (null: no gate), n the
+    // result's column: mul_col 1 is a gate an element, 0 one a row
+    const float* mul; long long mul_ld; int mul_col;
 };
+
+__device__ __forceinline__ float out_gate(const GemmParams& p, int t, int n) {
+    return p.mul ? 1.0f / (1.0f + __expf(-p.mul[(long long)t * p.mul_ld + (long long)n * p.mul_col])) : 1.0f;
+}
 
 __device__ __forceinline__ float unary_of(int kind, float v) {
     if (kind == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
@@ -124,7 +131,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
                     if (t >= p.T) break;
                     const float own = __uint_as_float(up ? r[8 + c] : r[c]), other = xch[col * 64 + fl];
                     const float g = up ? other : own, u = up ? own : other;
-                    out[(long long)t * p.ldo + f] = from_f32<TO>(gate_product(p, g, u));
+                    out[(long long)t * p.ldo + f] = from_f32<TO>(gate_product(p, g, u) * out_gate(p, t, f));
                 }
             }
             asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -135,14 +142,14 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
                 if (t >= p.T) break;
                 const float v = __uint_as_float(r[c]);
                 TO* dst = out + (long long)t * p.ldo + n;
-                if (EPI == EPI_STORE) *dst = from_f32<TO>(unary_of(p.unary, v));
+                if (EPI == EPI_STORE) *dst = from_f32<TO>(unary_of(p.unary, v) * out_gate(p, t, n));
                 else if (EPI == EPI_ADD) {
                     // a reduction at the memory side: no load, no wait; one writer an element
                     // unless K is split, so the sum's order is fixed in that case
                     asm volatile("red.global.add.f32 [%0], %1;" ::"l"(dst), "f"(v) : "memory");
                 } else {
                     const float u = __uint_as_float(r2[c]);
-                    *dst = from_f32<TO>(gate_product(p, v, u));
+                    *dst = from_f32<TO>(gate_product(p, v, u) * out_gate(p, t, n));
                 }
             }
         }
@@ -297,6 +304,7 @@ struct GroupParams {
     long long w_row_step;      // rows between two matrices in the weight map
     int a_col_step;            // batched: columns between two matrices' inputs in an activation row
     long long o_col_step;      // batched: columns between two matrices' outputs in an output row
+    int mul_mat_step;          // batched: columns between two matrices' gates in a row of ``mul``
 };
 
 template <int BN, int EPI, typename TO>
@@ -400,6 +408,7 @@ gemm_tc_grouped_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
             GemmParams pt = p;                           // this tile's rows end at t_end; matrix e's columns start at e * o_col_step
             pt.T = t_end;
             pt.out = (TO*)p.out + (long long)e * gp.o_col_step;
+            if (p.mul) pt.mul = p.mul + (long long)e * gp.mul_mat_step;
             epilogue_tile<BN, EPI, TO>(pt, tmem_base, q, lane, blockIdx.x, t0, 0, (float*)smem);
         }
     }
@@ -864,17 +873,19 @@ static int launch_bn(const CUtensorMap* mw, const CUtensorMap* mw2, const CUtens
 }
 
 // map_w (and map_w2 for EPI_SWIGLU): weights [N, K], boxes of 128 rows; map_a: activations [T, K],
-// boxes of ``bn`` rows.  ``gate`` (host, three floats or null): limit, alpha and shift of the gate product.
+// boxes of ``bn`` rows.  ``gate`` (host, three floats or null): limit, alpha and shift of the gate product.  ``mul`` (float32,
+// device, or null): the result times the sigmoid of mul[t * mul_ld + n * mul_col] (whole K, not with the adding epilogue).
 // splits > 1 cuts K into slices of kb_per_split blocks of 64: EPI_ADD then adds
 // with atomics, EPI_STORE (float32 only) writes slice z at out + z * split_stride.
 UB_API int ub_gemm_tc(const void* map_w, const void* map_w2, const void* map_a, void* out, int o_dtype, long long ldo,
                       long long split_stride, int T, int N, int K, int bn, int epi, int splits, int* error,
-                      const float* gate, cudaStream_t st) {
+                      const float* gate, const float* mul, long long mul_ld, int mul_col, cudaStream_t st) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || splits < 1) return UB_ERR_ARG;
     if (splits > 1 && (epi == EPI_SWIGLU || epi == EPI_SWIGLU_IL)) return UB_ERR_ARG;
     if (epi == EPI_SWIGLU_IL && (N % 128) != 0) return UB_ERR_ARG;
     if (splits > 1 && epi == EPI_STORE && o_dtype != UB_F32) return UB_ERR_ARG;
+    if (mul && (splits > 1 || epi == EPI_ADD)) return UB_ERR_ARG;
     const int nkb = (K + BK - 1) / BK;
     GemmParams p;
     p.out = out; p.ldo = ldo; p.split_stride = splits > 1 ? split_stride : 0;
@@ -884,6 +895,7 @@ UB_API int ub_gemm_tc(const void* map_w, const void* map_w2, const void* map_a, 
     p.share_tail = 0;
     p.error = error;
     set_gate_constants(p, gate);
+    p.mul = mul; p.mul_ld = mul_ld; p.mul_col = mul_col;
     if ((long long)(splits - 1) * p.kb_per_split >= nkb) return UB_ERR_ARG;      // an empty slice
     const CUtensorMap* mw = (const CUtensorMap*)map_w;
     const CUtensorMap* mw2 = (const CUtensorMap*)(map_w2 ? map_w2 : map_w);
@@ -940,17 +952,20 @@ static int launch_grouped_bn(const CUtensorMap* mw, const CUtensorMap* mw2, cons
 UB_API int ub_gemm_tc_grouped(const void* map_w, const void* map_w2, const void* map_a, void* out, int o_dtype, long long ldo,
                               int T, int N, int K, int bn, int epi, const void* tiles, const int* n_tiles, int max_tiles,
                               int n_mats, long long w_row_step, int a_col_step, long long o_col_step, int* error,
-                              const float* gate, cudaStream_t st) {
+                              const float* gate, const float* mul, long long mul_ld, int mul_col, int mul_mat_step, cudaStream_t st) {
     if (N <= 0 || (tiles ? max_tiles <= 0 : (T <= 0 || n_mats <= 0))) return 0;
     if (K <= 0 || (tiles && !n_tiles) || (a_col_step % 8) != 0) return UB_ERR_ARG;
     if (epi == EPI_SWIGLU && !map_w2) return UB_ERR_ARG;
+    if (mul && tiles) return UB_ERR_ARG;                   // (sorted rows are not the rows a gate is given for)
     GemmParams p;
     p.out = out; p.ldo = ldo; p.split_stride = 0;
     p.T = T; p.N = N; p.K = K;
     p.kb_per_split = (K + BK - 1) / BK;
     p.atomic = 0; p.share_tail = 0; p.error = error;
     set_gate_constants(p, gate);
+    p.mul = mul; p.mul_ld = mul_ld; p.mul_col = mul_col;
     GroupParams gp;
+    gp.mul_mat_step = mul_mat_step;
     gp.tiles = (const int4*)tiles; gp.n_tiles = n_tiles; gp.w_row_step = w_row_step; gp.a_col_step = a_col_step;
     gp.o_col_step = o_col_step;
     dim3 grid((N + BM - 1) / BM, tiles ? max_tiles : (T + bn - 1) / bn, tiles ? 1 : n_mats);
@@ -997,7 +1012,8 @@ static int launch_pair(const CUtensorMap* mw, const CUtensorMap* ma, GemmParams 
 }
 
 UB_API int ub_gemm_tc_pair(const void* map_w, const void* map_a, void* out, int o_dtype, long long ldo, int T, int N,
-                           int K, int epi, int* error, const float* gate, cudaStream_t st) {
+                           int K, int epi, int* error, const float* gate, const float* mul, long long mul_ld, int mul_col,
+                           cudaStream_t st) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0) return UB_ERR_ARG;
     if (epi == EPI_SWIGLU_IL && (N % 128) != 0) return UB_ERR_ARG;
@@ -1007,6 +1023,8 @@ UB_API int ub_gemm_tc_pair(const void* map_w, const void* map_a, void* out, int 
     p.kb_per_split = (K + BK - 1) / BK;
     p.atomic = 0; p.share_tail = 0; p.error = error;
     set_gate_constants(p, gate);
+    if (mul && epi == EPI_ADD) return UB_ERR_ARG;
+    p.mul = mul; p.mul_ld = mul_ld; p.mul_col = mul_col;
     const CUtensorMap* mw = (const CUtensorMap*)map_w;
     const CUtensorMap* ma = (const CUtensorMap*)map_a;
     if (epi == EPI_STORE && o_dtype == UB_BF16) return launch_pair<EPI_STORE, __nv_bfloat16>(mw, ma, p, st);

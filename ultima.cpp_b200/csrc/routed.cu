@@ -18,7 +18,10 @@
 //             identity expert), in the order of k.
 // ``mode`` (bits) and ``wscale`` choose another router of the same family: bit 0, s = sigmoid(z) instead of the softmax;
 // bit 1, a group's score is the sum of its two largest choice scores instead of the largest; bit 2, the chosen outputs'
-// weights are divided by their sum (+ 1e-20); the weights are then multiplied by ``wscale``.
+// weights are divided by their sum (+ 1e-20); bit 3, the scores are the logits themselves and the chosen outputs' weights are the
+// softmax over the chosen logits only; the weights are then multiplied by ``wscale``.
+// A row of z may have columns behind the router's outputs (another small product of the same input): ``extra`` receives the sum of
+// the K slices of the first of them.
 // Places within a segment are handed out by an atomic counter, so they differ from run to run; every row of a
 // product is computed on its own, so no result depends on them.
 #include "common.cuh"
@@ -39,7 +42,9 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
         sc[i] = v;
         m = fmaxf(m, v);
     }
-    if (mode & 1) {
+    if (mode & 8) {
+        for (int i = lane; i < n_out; i += 32) ch[i] = sc[i] + (corr ? corr[i] : 0.f);
+    } else if (mode & 1) {
         for (int i = lane; i < n_out; i += 32) { const float s = 1.0f / (1.0f + expf(-sc[i])); sc[i] = s; ch[i] = s + (corr ? corr[i] : 0.f); }
     } else {
         m = warp_max(m);
@@ -101,7 +106,12 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
         }
         __syncwarp();
     }
-    if (lane == 0 && ((mode & 4) || wscale != 1.0f)) {
+    if (lane == 0 && (mode & 8)) {
+        float top_z = -INFINITY, sum = 0.f;
+        for (int k = 0; k < top; ++k) top_z = fmaxf(top_z, wts_t[k]);
+        for (int k = 0; k < top; ++k) { const float e = expf(wts_t[k] - top_z); wts_t[k] = e; sum += e; }
+        for (int k = 0; k < top; ++k) wts_t[k] = wts_t[k] / sum * wscale;
+    } else if (lane == 0 && ((mode & 4) || wscale != 1.0f)) {
         float f = wscale;
         if (mode & 4) {
             float sum = 0.f;
@@ -112,10 +122,16 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
     }
 }
 
+__device__ __forceinline__ float extra_sum(const float* __restrict__ zr, int n_parts, long long part_stride, int n_out) {
+    float v = zr[n_out];
+    for (int s = 1; s < n_parts; ++s) v += zr[s * part_stride + n_out];
+    return v;
+}
+
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_kernel(const float* __restrict__ z, long long ldz, int n_parts, long long part_stride, const float* __restrict__ corr,
              int n_tokens, int n_out, int n_experts, int top, int n_groups, int keep, int* __restrict__ idx,
-             float* __restrict__ wts, int* __restrict__ counts, int mode, float wscale) {
+             float* __restrict__ wts, int* __restrict__ counts, int mode, float wscale, float* __restrict__ extra) {
     extern __shared__ float sm[];
     pdl_trigger();
     pdl_wait();
@@ -127,6 +143,7 @@ route_kernel(const float* __restrict__ z, long long ldz, int n_parts, long long 
     float* gm = ch + n_out;                                      // a group's best choice score
     route_token(z + t * ldz, n_parts, part_stride, corr, n_out, n_experts, top, n_groups, keep, sc, ch, gm, lane,
                 idx + t * top, wts + t * top, counts, mode, wscale);
+    if (extra && lane == 0) extra[t] = extra_sum(z + t * ldz, n_parts, part_stride, n_out);
 }
 
 // route, plan and scatter of a step of few tokens in ONE block (the counters live in shared memory; the global ones are
@@ -137,7 +154,7 @@ __global__ void __launch_bounds__(SMALL_WARPS * 32)
 route_small_kernel(const float* __restrict__ z, long long ldz, int n_parts, long long part_stride, const float* __restrict__ corr,
                    int n_tokens, int n_out, int n_experts, int top, int n_groups, int keep, int* __restrict__ idx,
                    float* __restrict__ wts, int4* __restrict__ tiles, int* __restrict__ n_tiles, int* __restrict__ row_pos,
-                   int* __restrict__ src_rows, int tile, int mode, float wscale) {
+                   int* __restrict__ src_rows, int tile, int mode, float wscale, float* __restrict__ extra) {
     extern __shared__ float sm[];
     pdl_trigger();
     pdl_wait();
@@ -153,6 +170,7 @@ route_small_kernel(const float* __restrict__ z, long long ldz, int n_parts, long
     for (int t = warp; t < n_tokens; t += SMALL_WARPS) {
         route_token(z + (long long)t * ldz, n_parts, part_stride, corr, n_out, n_experts, top, n_groups, keep, sc, sc + n_out,
                     sc + 2 * n_out, lane, idx + (long long)t * top, wts + (long long)t * top, cnt, mode, wscale);
+        if (extra && lane == 0) extra[t] = extra_sum(z + (long long)t * ldz, n_parts, part_stride, n_out);
         __syncwarp();
     }
     __syncthreads();
@@ -286,7 +304,7 @@ __global__ void combine_vec_kernel(const TY* __restrict__ y, const TH* __restric
 // whose sum they are.
 UB_API int ub_route(const float* z, long long ldz, int n_parts, long long part_stride, const float* corr, int n_tokens,
                     int n_out, int n_experts, int top, int n_groups, int keep, int* idx, float* wts, int* counts,
-                    int mode, float wscale, cudaStream_t st) {
+                    int mode, float wscale, float* extra, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     if (n_parts < 1) return UB_ERR_ARG;
     if (n_out < 1 || n_experts < 0 || n_experts > n_out || top < 1 || top > n_out || n_groups < 1 || n_out % n_groups ||
@@ -295,7 +313,7 @@ UB_API int ub_route(const float* z, long long ldz, int n_parts, long long part_s
     if (smem > 48 * 1024) return UB_ERR_ARG;
     const unsigned grid = (unsigned)((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS);
     return (int)ub_launch_dependent(route_kernel, dim3(grid), dim3(ROUTE_WARPS * 32), smem, st, z, ldz, n_parts, part_stride, corr,
-                                    n_tokens, n_out, n_experts, top, n_groups, keep, idx, wts, counts, mode, wscale);
+                                    n_tokens, n_out, n_experts, top, n_groups, keep, idx, wts, counts, mode, wscale, extra);
 }
 
 // The three steps above in one launch, for steps of at most ROUTE_SMALL_TOKENS tokens.
@@ -304,7 +322,7 @@ UB_API int ub_route_small_tokens() { return ROUTE_SMALL_TOKENS; }
 
 UB_API int ub_route_small(const float* z, long long ldz, int n_parts, long long part_stride, const float* corr, int n_tokens,
                           int n_out, int n_experts, int top, int n_groups, int keep, int* idx, float* wts, void* tiles,
-                          int* n_tiles, int* row_pos, int* src_rows, int tile, int mode, float wscale, cudaStream_t st) {
+                          int* n_tiles, int* row_pos, int* src_rows, int tile, int mode, float wscale, float* extra, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
     if (n_parts < 1 || n_tokens > ROUTE_SMALL_TOKENS || tile < 1) return UB_ERR_ARG;
     if (n_out < 1 || n_experts < 1 || n_experts > n_out || top < 1 || top > n_out || n_groups < 1 || n_out % n_groups ||
@@ -313,7 +331,7 @@ UB_API int ub_route_small(const float* z, long long ldz, int n_parts, long long 
     if (smem > 48 * 1024) return UB_ERR_ARG;
     return (int)ub_launch_dependent(route_small_kernel, dim3(1), dim3(SMALL_WARPS * 32), smem, st, z, ldz, n_parts, part_stride,
                                     corr, n_tokens, n_out, n_experts, top, n_groups, keep, idx, wts, (int4*)tiles, n_tiles,
-                                    row_pos, src_rows, tile, mode, wscale);
+                                    row_pos, src_rows, tile, mode, wscale, extra);
 }
 
 UB_API int ub_route_plan(int* counts, int* cursor, int* seg_start, void* tiles, int* n_tiles, int n_experts, int tile,

@@ -1,7 +1,9 @@
 // Row-wise kernels around a residual stream whose sublayers are scaled channel by channel and read their
 // input through a short convolution over time.
 //
-//   layernorm        (x - mean) / sqrt(var + eps) * w, the variance about the mean, no bias; float32 sums
+//   layernorm        (x - mean) / sqrt(var + eps) * w (+ b), the variance about the mean; float32 sums
+//   norm_join        x += mult * norm(y) with an RMS or a layer norm of the result's own, y cleared, and in the same pass the
+//                    next sublayer's input: nothing, x in the activation type, an RMS norm or a layer norm of the new x
 //   scale_add_norm   x += s * y (s one number a channel), y cleared, and in the same pass the next sublayer's
 //                    input: nothing, x in the activation type, an RMS norm or a layer norm of the new x
 //   causal_conv      y_t = sum_j w[:, j] u_(t - taps + 1 + j) for every channel of a projection row (the sum of K
@@ -23,7 +25,7 @@ __device__ __forceinline__ float rw_sigmoid(float x) { return 1.0f / (1.0f + exp
 
 // ---------------------------------------------------------------------------------------
 template <typename TO>
-__global__ void layernorm_kernel(const float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ out,
+__global__ void layernorm_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b, TO* __restrict__ out,
                                  const int* __restrict__ rows, int width, float eps) {
     __shared__ float red[33];
     pdl_trigger();
@@ -37,14 +39,14 @@ __global__ void layernorm_kernel(const float* __restrict__ x, const float* __res
     for (int i = threadIdx.x; i < width; i += blockDim.x) { const float d = xr[i] - mean; ss += d * d; }
     const float inv = inv_rms(block_sum(ss, red), (float)width, eps);
     TO* o = out + (long long)blockIdx.x * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>((xr[i] - mean) * inv * w[i]);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>((xr[i] - mean) * inv * w[i] + (b ? b[i] : 0.f));
 }
 
 // The same with a row held in registers: four neighbouring columns a load, one pass over global memory (rows of a
 // multiple of 4 columns, up to 256 * 4 * NCH of them).
 template <typename TO, int NCH>
 __global__ void __launch_bounds__(256)
-layernorm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, TO* __restrict__ out,
+layernorm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ b, TO* __restrict__ out,
                      const int* __restrict__ rows, int width, float eps) {
     __shared__ float red[33];
     pdl_trigger();
@@ -77,33 +79,37 @@ layernorm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, T
         const int c = threadIdx.x + i * 256;
         if (c < chunks) {
             const float4 ww = w4[c];
-            const float y[4] = {v[i].x * inv * ww.x, v[i].y * inv * ww.y, v[i].z * inv * ww.z, v[i].w * inv * ww.w};
+            float y[4] = {v[i].x * inv * ww.x, v[i].y * inv * ww.y, v[i].z * inv * ww.z, v[i].w * inv * ww.w};
+            if (b) {
+                const float4 bb = reinterpret_cast<const float4*>(b)[c];
+                y[0] += bb.x; y[1] += bb.y; y[2] += bb.z; y[3] += bb.w;
+            }
             store_vec<TO, 4>(o + 4 * c, y);
         }
     }
 }
 
-UB_API int ub_layernorm(const float* x, const float* w, void* out, int out_dtype, const int* rows, int n_rows, int width,
+UB_API int ub_layernorm(const float* x, const float* w, const float* b, void* out, int out_dtype, const int* rows, int n_rows, int width,
                         float eps, cudaStream_t st) {
     if (n_rows <= 0) return 0;
     if (width <= 0) return UB_ERR_ARG;
     if (out_dtype != UB_F32 && out_dtype != UB_BF16) return UB_ERR_UNSUPPORTED;
     cudaError_t e;
-    const bool aligned = (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0;
+    const bool aligned = (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
     if (width % 4 == 0 && width <= 256 * 4 * 8 && aligned) {
         const int nch = (width / 4 + 255) / 256;
 #define GO(NCH) e = out_dtype == UB_F32 \
-            ? ub_launch_dependent(layernorm_vec_kernel<float, NCH>, dim3(n_rows), dim3(256), 0, st, x, w, (float*)out, rows, width, eps) \
-            : ub_launch_dependent(layernorm_vec_kernel<__nv_bfloat16, NCH>, dim3(n_rows), dim3(256), 0, st, x, w, (__nv_bfloat16*)out, rows, width, eps)
+            ? ub_launch_dependent(layernorm_vec_kernel<float, NCH>, dim3(n_rows), dim3(256), 0, st, x, w, b, (float*)out, rows, width, eps) \
+            : ub_launch_dependent(layernorm_vec_kernel<__nv_bfloat16, NCH>, dim3(n_rows), dim3(256), 0, st, x, w, b, (__nv_bfloat16*)out, rows, width, eps)
         if (nch <= 1) GO(1); else if (nch <= 2) GO(2); else if (nch <= 4) GO(4); else GO(8);
 #undef GO
         return (int)e;
     }
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     if (out_dtype == UB_F32)
-        e = ub_launch_dependent(layernorm_kernel<float>, dim3(n_rows), dim3(threads), 0, st, x, w, (float*)out, rows, width, eps);
+        e = ub_launch_dependent(layernorm_kernel<float>, dim3(n_rows), dim3(threads), 0, st, x, w, b, (float*)out, rows, width, eps);
     else
-        e = ub_launch_dependent(layernorm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, x, w, (__nv_bfloat16*)out, rows, width, eps);
+        e = ub_launch_dependent(layernorm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, x, w, b, (__nv_bfloat16*)out, rows, width, eps);
     return (int)e;
 }
 
@@ -111,7 +117,7 @@ UB_API int ub_layernorm(const float* x, const float* w, void* out, int out_dtype
 // mode: 0 nothing goes out, 1 the new x as it is, 2 its RMS norm times nw, 3 its layer norm times nw
 template <typename TO>
 __global__ void scale_add_norm_kernel(float* __restrict__ y, const float* __restrict__ scale, float* __restrict__ x, int mode,
-                                      const float* __restrict__ nw, float eps, TO* __restrict__ out, int width, int clear_y) {
+                                      const float* __restrict__ nw, const float* __restrict__ nb, float eps, TO* __restrict__ out, int width, int clear_y) {
     __shared__ float red[33];
     pdl_trigger();
     pdl_wait();
@@ -139,20 +145,154 @@ __global__ void scale_add_norm_kernel(float* __restrict__ y, const float* __rest
         for (int i = threadIdx.x; i < width; i += blockDim.x) { const float d = xr[i] - mean; ss += d * d; }
     }
     const float inv = inv_rms(block_sum(ss, red), (float)width, eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>((xr[i] - mean) * inv * nw[i]);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>((xr[i] - mean) * inv * nw[i] + (nb ? nb[i] : 0.f));
 }
 
-UB_API int ub_scale_add_norm(float* y, const float* scale, float* x, int mode, const float* nw, float eps, void* out,
+UB_API int ub_scale_add_norm(float* y, const float* scale, float* x, int mode, const float* nw, const float* nb, float eps, void* out,
                              int out_dtype, int n_rows, int width, int clear_y, cudaStream_t st) {
     if (n_rows <= 0) return 0;
     if (width <= 0 || mode < 0 || mode > 3 || (mode >= 2 && !nw) || (mode >= 1 && !out)) return UB_ERR_ARG;
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     cudaError_t e;
     if (mode == 0 || out_dtype == UB_F32)
-        e = ub_launch_dependent(scale_add_norm_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y, scale, x, mode, nw, eps, (float*)out, width, clear_y);
+        e = ub_launch_dependent(scale_add_norm_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y, scale, x, mode, nw, nb, eps, (float*)out, width, clear_y);
     else if (out_dtype == UB_BF16)
-        e = ub_launch_dependent(scale_add_norm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y, scale, x, mode, nw, eps, (__nv_bfloat16*)out, width, clear_y);
+        e = ub_launch_dependent(scale_add_norm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y, scale, x, mode, nw, nb, eps, (__nv_bfloat16*)out, width, clear_y);
     else return UB_ERR_UNSUPPORTED;
+    return (int)e;
+}
+
+// ---------------------------------------------------------------------------------------
+// x += mult * norm_a(y), y cleared, out = what ``mode`` names of the new x (0 nothing, 1 x as it is, 2 an RMS norm, 3 a layer
+// norm).  norm_a: a layer norm (``a_layer``) or an RMS norm.  Every norm is (v - mean) * inv * w + b with mean 0 for the RMS
+// norms and no b where the pointer is null.
+struct JoinNorm { const float* w; const float* b; float eps; int layer; };
+
+template <typename TO>
+__global__ void norm_join_kernel(float* __restrict__ y, float* __restrict__ x, float mult, JoinNorm a, int mode, JoinNorm n,
+                                 TO* __restrict__ out, int width, int clear_y) {
+    __shared__ float red[33];
+    pdl_trigger();
+    pdl_wait();
+    float* yr = y + (long long)blockIdx.x * width;
+    float* xr = x + (long long)blockIdx.x * width;
+    auto stats = [&](const float* v, bool layer, float eps, float& mean, float& inv) {
+        mean = 0.f;
+        if (layer) {
+            float s = 0.f;
+            for (int i = threadIdx.x; i < width; i += blockDim.x) s += v[i];
+            mean = block_sum(s, red) / (float)width;
+        }
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) { const float d = v[i] - mean; ss += d * d; }
+        inv = inv_rms(block_sum(ss, red), (float)width, eps);
+    };
+    float mean, inv;
+    stats(yr, a.layer, a.eps, mean, inv);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {          // (a thread meets its own elements only, here and below)
+        xr[i] = fmaf(mult, (yr[i] - mean) * inv * a.w[i] + (a.b ? a.b[i] : 0.f), xr[i]);
+        if (clear_y) yr[i] = 0.f;
+    }
+    if (mode == 0) return;
+    TO* o = out + (long long)blockIdx.x * width;
+    if (mode == 1) {
+        for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>(xr[i]);
+        return;
+    }
+    stats(xr, mode == 3, n.eps, mean, inv);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_f32<TO>((xr[i] - mean) * inv * n.w[i] + (n.b ? n.b[i] : 0.f));
+}
+
+// The same with both rows in registers, four neighbouring columns a load (rows of a multiple of 4 columns, up to 256 * 4 * NCH).
+template <typename TO, int NCH>
+__global__ void __launch_bounds__(256)
+norm_join_vec_kernel(float* __restrict__ y, float* __restrict__ x, float mult, JoinNorm a, int mode, JoinNorm n,
+                     TO* __restrict__ out, int width, int clear_y) {
+    __shared__ float red[33];
+    pdl_trigger();
+    pdl_wait();
+    float4* yr = reinterpret_cast<float4*>(y + (long long)blockIdx.x * width);
+    float4* xr = reinterpret_cast<float4*>(x + (long long)blockIdx.x * width);
+    const int chunks = width >> 2;
+    float4 v[NCH], u[NCH];
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = threadIdx.x + i * 256;
+        v[i] = c < chunks ? yr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+        u[i] = c < chunks ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    // the row's mean taken off (layer norm), and 1 / sqrt(mean square + eps) of what is left; columns past the row stay zero
+    auto centred = [&](float4* r, bool layer, float eps) -> float {
+        if (layer) {
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < NCH; ++i) s += (r[i].x + r[i].y) + (r[i].z + r[i].w);
+            const float mean = block_sum(s, red) / (float)width;
+#pragma unroll
+            for (int i = 0; i < NCH; ++i)
+                if (threadIdx.x + i * 256 < chunks) { r[i].x -= mean; r[i].y -= mean; r[i].z -= mean; r[i].w -= mean; }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) ss += (r[i].x * r[i].x + r[i].y * r[i].y) + (r[i].z * r[i].z + r[i].w * r[i].w);
+        return inv_rms(block_sum(ss, red), (float)width, eps);
+    };
+    auto scaled = [](const float4& r, float inv, const float* w, const float* b, int c) -> float4 {
+        const float4 ww = reinterpret_cast<const float4*>(w)[c];
+        float4 o = make_float4(r.x * inv * ww.x, r.y * inv * ww.y, r.z * inv * ww.z, r.w * inv * ww.w);
+        if (b) {
+            const float4 bb = reinterpret_cast<const float4*>(b)[c];
+            o.x += bb.x; o.y += bb.y; o.z += bb.z; o.w += bb.w;
+        }
+        return o;
+    };
+    float inv = centred(v, a.layer, a.eps);
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < chunks) {
+            const float4 d = scaled(v[i], inv, a.w, a.b, c);
+            u[i].x = fmaf(mult, d.x, u[i].x); u[i].y = fmaf(mult, d.y, u[i].y);
+            u[i].z = fmaf(mult, d.z, u[i].z); u[i].w = fmaf(mult, d.w, u[i].w);
+            xr[c] = u[i];
+            if (clear_y) yr[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    if (mode == 0) return;
+    TO* o = out + (long long)blockIdx.x * width;
+    if (mode >= 2) inv = centred(u, mode == 3, n.eps);
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < chunks) {
+            const float4 r = mode >= 2 ? scaled(u[i], inv, n.w, n.b, c) : u[i];
+            const float e[4] = {r.x, r.y, r.z, r.w};
+            store_vec<TO, 4>(o + 4 * c, e);
+        }
+    }
+}
+
+UB_API int ub_norm_join(float* y, float* x, float mult, const float* aw, const float* ab, float a_eps, int a_layer, int mode,
+                        const float* nw, const float* nb, float n_eps, void* out, int out_dtype, int n_rows, int width, int clear_y,
+                        cudaStream_t st) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0 || !aw || mode < 0 || mode > 3 || (mode >= 2 && !nw) || (mode >= 1 && !out)) return UB_ERR_ARG;
+    if (mode >= 1 && out_dtype != UB_F32 && out_dtype != UB_BF16) return UB_ERR_UNSUPPORTED;
+    const JoinNorm a{aw, ab, a_eps, a_layer ? 1 : 0}, n{nw, nb, n_eps, mode == 3 ? 1 : 0};
+    const bool f32 = mode == 0 || out_dtype == UB_F32;
+    const bool aligned = (((uintptr_t)x | (uintptr_t)y | (uintptr_t)aw | (uintptr_t)ab | (uintptr_t)nw | (uintptr_t)nb | (uintptr_t)out) & 15) == 0;
+    cudaError_t e;
+    if (width % 4 == 0 && width <= 256 * 4 * 8 && aligned) {
+        const int nch = (width / 4 + 255) / 256;
+#define GO(NCH) e = f32 ? ub_launch_dependent(norm_join_vec_kernel<float, NCH>, dim3(n_rows), dim3(256), 0, st, y, x, mult, a, mode, n, (float*)out, width, clear_y) \
+                        : ub_launch_dependent(norm_join_vec_kernel<__nv_bfloat16, NCH>, dim3(n_rows), dim3(256), 0, st, y, x, mult, a, mode, n, (__nv_bfloat16*)out, width, clear_y)
+        if (nch <= 1) GO(1); else if (nch <= 2) GO(2); else if (nch <= 4) GO(4); else GO(8);
+#undef GO
+        return (int)e;
+    }
+    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+    e = f32 ? ub_launch_dependent(norm_join_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y, x, mult, a, mode, n, (float*)out, width, clear_y)
+            : ub_launch_dependent(norm_join_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y, x, mult, a, mode, n, (__nv_bfloat16*)out, width, clear_y);
     return (int)e;
 }
 

@@ -95,6 +95,9 @@ class Model:
                 raise ValueError(f"run list names layer {r.layer}; the model has {len(self.layers)}")
             if r.entry is not None and not (0 <= r.entry < len(self.entries)):
                 raise ValueError(f"run list names entry {r.entry}; the model has {len(self.entries)}")
+        # for each run the layer that reads the stream right behind it, or None (the end, or an entry in between): an arrangement
+        # may prepare that layer's input in its own last kernel
+        self._following = [self.layers[b.layer] if b.entry is None else None for b in spec.runs[1:]] + [None]
         self._keeps_embedding = any(self.entries[r.entry].needs_embedding_output for r in spec.runs if r.entry is not None)
         # an embedding that keeps per-sequence state gets a place in the cache behind the runs'
         need = getattr(self.embedding, "cache_need", None)
@@ -161,6 +164,7 @@ class Model:
                 layer = self.layers[r.layer]
                 if r.entry is not None:
                     self.entries[r.entry].forward(x, x0, rt)
+                rt.next_layer = self._following[i]
                 layer.arrangement.run(layer, x, batch, cache.run_cache(i, batch.tables), rt)
                 if TRACE:
                     _trace("l_out", i, x)

@@ -89,6 +89,7 @@ class Runtime:
         self.launches = 0              # kernels of this library launched through the runtime
         self.pass_id = 0               # counts the passes through the layers (Model.forward); what an arrangement
                                        # keeps from layer to layer is valid within one pass only
+        self.next_layer = None         # the layer that reads the stream behind the one that is running (set by Model.forward)
         # flags the kernels raise: [0] a token id outside the vocabulary, [1] a wait that ran out
         # (they are the head of a buffer whose tail takes the sampled token ids: one copy brings both)
         self.status_and_ids = torch.zeros(4 + 4096, dtype=torch.int32, device=self.device)
@@ -123,11 +124,12 @@ class Runtime:
             raise RuntimeError("a wait inside a kernel ran out of time; the step's results are not valid")
 
     # ---- products ----------------------------------------------------------------------
-    def matmul(self, a, w, out, epilogue=ops.EPI_STORE, w2=None, gate=None, unary=0):
+    def matmul(self, a, w, out, epilogue=ops.EPI_STORE, w2=None, gate=None, unary=0, mul=None):
         """out (=, +=) a @ w.T with float32 accumulation; see kernels.ops for the epilogues.  ``gate`` =
         (limit, alpha, shift): the constants of a clamped gate product (tensor-core epilogues only).  ``unary``
         (ops.UNARY_*): out = f(a @ w.T), the function taken of the float32 sums: in the tensor-core product's storing
-        epilogue, elsewhere by a kernel behind the product."""
+        epilogue, elsewhere by a kernel behind the product.  ``mul`` = (gates, column step): the stored result times a sigmoid
+        gate (see ``gemm_tc.mul_args``; tensor-core epilogues only)."""
         self.launches += 1
         if unary and (epilogue != ops.EPI_STORE or gate is not None):
             raise ops.KernelError("a function of the sums goes with the storing epilogue")
@@ -135,18 +137,18 @@ class Runtime:
             from ..kernels import gemm_tc
             if unary:
                 gate = gemm_tc.unary_constants(unary)
-            key = gemm_tc.launch_key(a, w, out, epilogue, w2, self._status_ptr, gate)
+            key = gemm_tc.launch_key(a, w, out, epilogue, w2, self._status_ptr, gate, mul)
             if gemm_tc.relaunch(key):
                 return None
             if gemm_tc.accepts(a, w, out, epilogue, w2):
-                return gemm_tc.gemm(a, w, out, epilogue, w2, self, key=key, gate=gate)
+                return gemm_tc.gemm(a, w, out, epilogue, w2, self, key=key, gate=gate, mul=mul)
         if unary:
             sums = self.arena.alloc(tuple(out.shape), torch.float32)
             ops.gemm_simt(a, w, sums)
             self.launches += 1
             return ops.unary(sums, out, unary)
-        if gate is not None:
-            raise ops.KernelError("a clamped gate product is an epilogue of the tensor-core product only")
+        if gate is not None or mul is not None:
+            raise ops.KernelError("a clamped gate product, or a gate on the result, is an epilogue of the tensor-core product only")
         if epilogue == ops.EPI_SWIGLU_IL:
             raise ops.KernelError("the interleaved gate/up layout is for the tensor-core product only; "
                                   "this call does not fit it (operand alignment)")
@@ -170,25 +172,35 @@ class Runtime:
         gemm_tc.gemm(a, w, out, ops.EPI_STORE, None, self, splits=parts)
         return out
 
-    def matmul_heads(self, a, w, out):
+    def matmul_heads(self, a, w, out, gate=None):
         """out[:, b, :] = a[:, b, :] @ w[b].T for every b (one small matrix a head): a [T, B, K], w [B, N, K], out
-        [T, B, N]; a and out may be column ranges of wider rows."""
+        [T, B, N]; a and out may be column ranges of wider rows.  ``gate`` float32 [T, B] or [T, B * N] (any row stride): the
+        result times its sigmoid, a number a matrix or an element, in the tensor-core product's epilogue or behind the product
+        (out is then contiguous)."""
         self.launches += 1
         if self.use_tensor_cores and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
             from ..kernels import gemm_tc
             if gemm_tc.accepts_batched(a, w, out):
-                return gemm_tc.batched(a, w, out, self)
-        return ops.gemm_batched(a, w, out)
+                return gemm_tc.batched(a, w, out, self, gate=gate)
+        ops.gemm_batched(a, w, out)
+        if gate is not None:
+            T, B, N = out.shape
+            self.launches += 1
+            if gate.shape[1] == B * N:
+                ops.elem_gate(out.view(T, B * N), gate)
+            else:
+                ops.head_gate(out.view(T, B * N), gate, B, N)
 
-    def matmul_grouped(self, a, w, out, plan, epilogue=ops.EPI_STORE, w2=None, unary=0):
+    def matmul_grouped(self, a, w, out, plan, epilogue=ops.EPI_STORE, w2=None, unary=0, gate=None):
         """Sorted rows against the matrix their tile names (``plan``: a routed feed-forward's ``RoutePlan``):
         out[p] = a[plan.src_rows[p] or p] @ w[e].T, e the expert of the tile that holds sorted row p.  The tensor-core
         product takes rows that lie in the sorted order already (``plan.gather`` False); ``grouped_on_tensor_cores``
-        says beforehand whether it will take a product.  ``unary`` (ops.UNARY_*): out = f(product), as in ``matmul``."""
+        says beforehand whether it will take a product.  ``unary`` (ops.UNARY_*): out = f(product), as in ``matmul``; ``gate`` =
+        (limit, alpha, shift): the constants of a clamped gate product."""
         self.launches += 1
         if not plan.gather and self.grouped_on_tensor_cores(a, w, out, epilogue, w2):
             from ..kernels import gemm_tc
-            return gemm_tc.grouped(a, w, out, plan, epilogue, w2, self, unary=unary)
+            return gemm_tc.grouped(a, w, out, plan, epilogue, w2, self, unary=unary, gate=gate)
         if unary:
             sums = self.arena.alloc(tuple(out.shape), torch.float32)
             ops.gemm_grouped(a, w, sums, plan.tiles, plan.n_tiles, plan.src_rows if plan.gather else None, plan.max_tiles,
@@ -196,7 +208,7 @@ class Runtime:
             self.launches += 1
             return ops.unary(sums, out, unary)
         return ops.gemm_grouped(a, w, out, plan.tiles, plan.n_tiles, plan.src_rows if plan.gather else None, plan.max_tiles,
-                                epilogue, w2)
+                                epilogue, w2, gate=gate)
 
     def grouped_on_tensor_cores(self, a, w, out, epilogue=ops.EPI_STORE, w2=None) -> bool:
         if not (self.use_tensor_cores and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16):
@@ -205,9 +217,9 @@ class Runtime:
         return gemm_tc.accepts_grouped(a, w, out, epilogue, w2)
 
     # ---- attention ----------------------------------------------------------------------
-    def attention_latent(self, q_lat, kv, batch, n_heads, row, rank, scale, window):
+    def attention_latent(self, q_lat, kv, batch, n_heads, row, rank, scale, window, sink_vals=None):
         """Attention of ``n_heads`` query heads [T, heads, row] over ONE key head whose rows [row] also hold the values
-        (their leading ``rank`` columns).  Returns the heads' weighted sums as a view [T, heads, rank] (of a wider
+        (their leading ``rank`` columns); ``sink_vals`` float32 [heads]: the softmax's sum has one more term exp(sink).  Returns the heads' weighted sums as a view [T, heads, rank] (of a wider
         buffer where the kernel returns whole rows)."""
         T = q_lat.shape[0]
         q2 = q_lat.view(T, n_heads * row)
@@ -216,11 +228,15 @@ class Runtime:
             from ..kernels import attn_tc
             if attn_tc.accepts(q2, kv, row, n_heads, 1) and attn_tc.LATENT:
                 o = self.arena.alloc((T, n_heads, row), self.dtype)
-                attn_tc.attention(q2, kv, o.view(T, n_heads * row), batch, n_heads, 1, row, scale, self, kernel="mma")
+                o2 = o.view(T, n_heads * row)
+                if sink_vals is not None:
+                    attn_tc.attention_ext(q2, kv, o2, batch, n_heads, 1, row, scale, self, window=window, sink=True, sink_vals=sink_vals)
+                else:
+                    attn_tc.attention(q2, kv, o2, batch, n_heads, 1, row, scale, self, kernel="mma")
                 return o[:, :, :rank]
         o = self.arena.alloc((T, n_heads, rank), self.dtype)
         ops.attn_simple(q2, kv.k, kv.k, o.view(T, n_heads * rank), batch.tok_pos, batch.tok_seq, kv.table, kv.ring, kv.page,
-                        n_heads, 1, row, window, scale, v_head_dim=rank, v_row=row)
+                        n_heads, 1, row, window, scale, v_head_dim=rank, v_row=row, sink=sink_vals is not None, sink_vals=sink_vals)
         return o
 
     def attention_from_qkv(self, qkv_parts, q_norm, k_norm, cos, sin, eps, kv, out, batch, n_heads, n_kv_heads,

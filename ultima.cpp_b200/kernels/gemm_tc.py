@@ -27,14 +27,14 @@ def lib():
         L.ub_tmap_bf16_2d.argtypes = [c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_int]
         L.ub_tmap_bf16_2d.restype = c_int
         L.ub_gemm_tc.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong,
-                                 c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]
+                                 c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p]
         L.ub_gemm_tc.restype = c_int
         L.ub_gemm_tc_pair.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int,
-                                      c_void_p, c_void_p, c_void_p]
+                                      c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p]
         L.ub_gemm_tc_pair.restype = c_int
         L.ub_gemm_tc_grouped.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int,
                                          c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_int, c_longlong, c_void_p,
-                                         c_void_p, c_void_p]
+                                         c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p]
         L.ub_gemm_tc_grouped.restype = c_int
         L.ub_gemm_tc_set_pdl.argtypes = [c_int]
         L.ub_gemm_tc_set_pdl.restype = None
@@ -142,11 +142,22 @@ def pairs(T: int, N: int, splits: int, epilogue: int, n_sms: int | None = None) 
     return -(-N // 256) * -(-T // 256) >= (n_sms or sm_count()) // 2
 
 
-def gemm(a, w, out, epilogue, w2, rt, splits: int | None = None, bn: int | None = None, key=None, gate=None):
+def mul_args(mul):
+    """A sigmoid gate on a stored result, ``mul`` = (gates, column step): gates float32 whose row t (any stride) belongs to
+    result row t; step 1: column n has gate n; step 0: one gate a row.  -> (pointer, row stride, column step)."""
+    if mul is None:
+        return 0, 0, 0
+    g, step = mul
+    assert g.dtype == torch.float32 and (g.dim() == 1 or g.stride(-1) == 1)
+    return g.data_ptr(), g.stride(0), int(step)
+
+
+def gemm(a, w, out, epilogue, w2, rt, splits: int | None = None, bn: int | None = None, key=None, gate=None, mul=None):
     """out: [T, N]; for EPI_SWIGLU_IL [T, N / 2]; for EPI_STORE with ``splits`` > 1 a float32
     [splits, T, N] whose sum over the first axis is the product.  ``gate`` = (limit, alpha, shift): the gate
     product of the two SWIGLU epilogues becomes g' sigmoid(alpha g') (u' + shift) with g' = min(g, limit) and
-    u' = clamp(u, -limit, limit); None: silu(g) u.  A fourth number is EPI_STORE's function of the sum (see ``unary_constants``)."""
+    u' = clamp(u, -limit, limit); None: silu(g) u.  A fourth number is EPI_STORE's function of the sum (see ``unary_constants``).
+    ``mul``: see ``mul_args``."""
     T, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(-1) == 1
@@ -167,13 +178,13 @@ def gemm(a, w, out, epilogue, w2, rt, splits: int | None = None, bn: int | None 
         fn, what = L.ub_gemm_tc_pair, "gemm_tc_pair"
         maps = (_tmap_entry(w, 128), _tmap_entry(a, 128))
         args = (maps[0][1], maps[1][1], _ptr(out), BF16 if out.dtype == torch.bfloat16 else F32,
-                out.stride(0), T, N, K, epilogue, _ptr(rt.status[1:2]), consts)
+                out.stride(0), T, N, K, epilogue, _ptr(rt.status[1:2]), consts, *mul_args(mul))
     else:
         fn, what = L.ub_gemm_tc, "gemm_tc"
         maps = (_tmap_entry(w, 128), _tmap_entry(w2, 128) if w2 is not None else (None, 0), _tmap_entry(a, bn))
         args = (maps[0][1], maps[1][1], maps[2][1], _ptr(out),
                 BF16 if out.dtype == torch.bfloat16 else F32, ldo, split_stride, T, N, K, bn, epilogue, s,
-                _ptr(rt.status[1:2]), consts)
+                _ptr(rt.status[1:2]), consts, *mul_args(mul))
     if key is not None:
         if len(_plans) > 8192:
             _plans.clear()
@@ -187,13 +198,13 @@ def gemm(a, w, out, epilogue, w2, rt, splits: int | None = None, bn: int | None 
 _plans: dict = {}
 
 
-def launch_key(a, w, out, epilogue, w2, status_ptr: int, gate=None):
+def launch_key(a, w, out, epilogue, w2, status_ptr: int, gate=None, mul=None):
     """Everything a plan depends on: places, shapes and strides of the operands and of the result, the
     epilogue, and the status word the kernel reports to (another engine's tensors may come to lie at the
     same addresses with other shapes)."""
     return (a.data_ptr(), a.shape[0], a.shape[1], a.stride(0), w.data_ptr(), w.shape[0], w.stride(0), out.data_ptr(),
             out.dim(), out.shape[-1], out.stride(-2) if out.dim() > 1 else 0, out.dtype, epilogue,
-            0 if w2 is None else w2.data_ptr(), status_ptr, USE_PAIRS, gate)
+            0 if w2 is None else w2.data_ptr(), status_ptr, USE_PAIRS, gate, mul_args(mul))
 
 
 def relaunch(key) -> bool:
@@ -266,17 +277,18 @@ def unary_constants(kind: int):
     return (float("inf"), 1.0, 0.0, float(kind))
 
 
-def grouped(a, w, out, plan, epilogue, w2, rt, unary: int = 0):
+def grouped(a, w, out, plan, epilogue, w2, rt, unary: int = 0, gate=None):
     """out[p] = a[p] @ w[e].T for the sorted rows p of every tile (e, first row, rows) of ``plan``; a [rows, K] lies in
-    the sorted order already.  ``plan.tile`` is the most rows a tile has (16 to 128)."""
+    the sorted order already.  ``plan.tile`` is the most rows a tile has (16 to 128).  ``gate``: constants of the gate product."""
     E, N, K = w.shape
     wv, step = _stacked(w)
     m2 = _tmap(_stacked(w2)[0], 128) if w2 is not None else 0
     bn = int(plan.tile)
+    consts = unary_constants(unary) if unary else tuple(gate) + (0.0,) if gate is not None else None
     rc = lib().ub_gemm_tc_grouped(_tmap(wv, 128), m2, _tmap(a, bn), _ptr(out), BF16 if out.dtype == torch.bfloat16 else F32,
                                   out.stride(0), a.shape[0], N, K, bn, epilogue, _ptr(plan.tiles), _ptr(plan.n_tiles),
                                   int(plan.max_tiles), E, step, 0, 0, _ptr(rt.status[1:2]),
-                                  (ctypes.c_float * 4)(*unary_constants(unary)) if unary else None, _stream())
+                                  (ctypes.c_float * 4)(*consts) if consts is not None else None, 0, 0, 0, 0, _stream())
     _check(rc, "gemm_tc_grouped")
 
 
@@ -289,15 +301,19 @@ def accepts_batched(a, w, out) -> bool:
             and out.dtype in (torch.bfloat16, torch.float32))
 
 
-def batched(a, w, out, rt):
-    """out[:, b, :] = a[:, b, :] @ w[b].T: a [T, B, K] and out [T, B, N] may be column ranges of wider rows."""
+def batched(a, w, out, rt, gate=None):
+    """out[:, b, :] = a[:, b, :] @ w[b].T: a [T, B, K] and out [T, B, N] may be column ranges of wider rows.  ``gate`` float32
+    [T, B] or [T, B * N]: the result times its sigmoid, a number a matrix or an element."""
     T, B, K = a.shape
     N = w.shape[1]
     wv, step = _stacked(w)
     a2 = torch.as_strided(a, (T, (B - 1) * a.stride(1) + K), (a.stride(0), 1))
     bn = token_tile(T, EPI_STORE)
     bn = min(bn, 128)
+    wide = gate is not None and gate.shape[1] == B * N and N != 1
+    assert gate is None or gate.shape == (T, B * N if wide else B)
     rc = lib().ub_gemm_tc_grouped(_tmap(wv, 128), 0, _tmap(a2, bn), _ptr(out), BF16 if out.dtype == torch.bfloat16 else F32,
                                   out.stride(0), T, N, K, bn, EPI_STORE, None, None, 0, B, step, a.stride(1), out.stride(1),
-                                  _ptr(rt.status[1:2]), None, _stream())
+                                  _ptr(rt.status[1:2]), None, *mul_args(None if gate is None else (gate, 1 if wide else 0)),
+                                  N if wide else 1, _stream())
     _check(rc, "gemm_tc_batched")

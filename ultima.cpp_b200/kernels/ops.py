@@ -97,14 +97,14 @@ def _declare(lib, source: str) -> None:
     P, I, L, F, U = c_void_p, c_int, c_longlong, c_float, c_ulonglong
     sigs = {
         "basic.cu": {
-            "ub_embed": [P, I, P, P, I, I, I, P, P],
+            "ub_embed": [P, I, P, P, I, I, I, P, F, P],
             "ub_rmsnorm": [P, P, P, P, I, I, I, F, P],
             "ub_qk_prepare": [P, I, I, L, P, I, L, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, I, I, P, P, L, P],
             "ub_rotate_pairs": [P, I, L, I, I, I, P, P, P, I, I, P],
             "ub_kv_write": [P, P, I, L, P, P, P, P, I, P, I, I, I, I, I, I, P],
             "ub_silu_mul": [P, I, I, L, P, I, I, I, P],
             "ub_rmsnorm_add": [P, P, P, P, I, I, I, F, I, P],
-            "ub_glu_clamped": [P, I, P, I, I, I, F, F, F, P],
+            "ub_glu_clamped": [P, I, P, I, I, I, F, F, F, P, L, P],
             "ub_head_gate": [P, I, L, P, L, I, I, I, P],
             "ub_convert": [P, I, P, I, L, P],
             "ub_add_into": [P, P, I, L, P],
@@ -116,16 +116,16 @@ def _declare(lib, source: str) -> None:
         },
         "gemm_simt.cu": {"ub_gemm_simt": [P, I, P, P, I, P, I, I, I, I, L, L, L, I, P],
                          "ub_gemm_simt_batched": [P, I, P, I, P, I, I, I, I, L, L, L, I, L, L, L, P],
-                         "ub_gemm_simt_grouped": [P, I, P, P, I, P, I, I, I, L, L, L, L, P, P, P, I, I, P]},
+                         "ub_gemm_simt_grouped": [P, I, P, P, I, P, I, I, I, L, L, L, L, P, P, P, I, I, P, P]},
         "streams.cu": {"ub_streams_fill": [P, P, I, I, I, P],
                        "ub_streams_pass": [P, L, I, P, P, P, P, I, P, P, P, I, I, I, F, P]},
-        "routed.cu": {"ub_route": [P, L, I, L, P, I, I, I, I, I, I, P, P, P, I, F, P],
+        "routed.cu": {"ub_route": [P, L, I, L, P, I, I, I, I, I, I, P, P, P, I, F, P, P],
                       "ub_route_plan": [P, P, P, P, P, I, I, P],
                       "ub_route_scatter": [P, P, P, P, P, I, I, I, P],
-                      "ub_route_small": [P, L, I, L, P, I, I, I, I, I, I, P, P, P, P, P, P, I, I, F, P],
+                      "ub_route_small": [P, L, I, L, P, I, I, I, I, I, I, P, P, P, P, P, P, I, I, F, P, P],
                       "ub_route_combine": [P, I, P, I, P, P, P, I, I, I, P],
                       "ub_route_gather": [P, P, P, I, I, L, P]},
-        "latent.cu": {"ub_latent_place": [P, I, L, I, L, I, I, P, P, I, P, P, P, I, P, P, P, I, P, I, I, I, I, I, I, I, I, F, P]},
+        "latent.cu": {"ub_latent_place": [P, I, L, I, L, I, P, I, P, I, P, P, I, I, P, P, P, I, P, I, I, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P]},
         "attn_simple.cu": {"ub_attn_simple": [P, L, I, P, P, I, P, L, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, L, I, P, I, I, F, F, P, I, P, I, P],
                            "ub_qkv_place_rows": [P, I, L, I, L, I, I, I, P, I, L, P, P, I, P, P, I, I, P, P, P, P, I, P, I, I, I, I, I,
                                                  I, I, I, F, I, I, P, P],
@@ -142,8 +142,9 @@ def _declare(lib, source: str) -> None:
                    "ub_ssm_finish": [P, P, L, I, L, P, P, P, I, I, I, F, F, P],
                    "ub_mamba1_scan": [P, I, P, P, P, L, I, I, P, P, P, L, I, L, P, I, P, P, P, I, I, I, I, P],
                    "ub_mamba1_scan_staged": [P, I, P, P, P, L, I, I, P, P, P, L, I, L, P, I, P, P, P, I, I, I, I, P, P]},
-        "rowwise.cu": {"ub_layernorm": [P, P, P, I, P, I, I, F, P],
-                       "ub_scale_add_norm": [P, P, P, I, P, F, P, I, I, I, I, P],
+        "rowwise.cu": {"ub_layernorm": [P, P, P, P, I, P, I, I, F, P],
+                       "ub_norm_join": [P, P, F, P, P, F, I, I, P, P, F, P, I, I, I, I, P],
+                       "ub_scale_add_norm": [P, P, P, I, P, P, F, P, I, I, I, I, P],
                        "ub_causal_conv": [P, I, L, I, L, I, P, P, P, I, P, P, P, P, I, L, I, I, I, I, I, I, I, I, P, P, P, P],
                        "ub_causal_conv_state": [P, I, L, I, L, I, P, P, P, P, I, I, I, P],
                        "ub_take_cols": [P, L, I, L, I, I, I, P, I, L, I, I, P],
@@ -158,14 +159,14 @@ def _declare(lib, source: str) -> None:
 
 
 # ---------------------------------------------------------------------------------------
-def embed(table, ids, out, status):
-    """out[t, :] = table[ids[t], :] as float32; a bad id raises ``status`` (int32[1])."""
+def embed(table, ids, out, status, scale=1.0):
+    """out[t, :] = scale * table[ids[t], :] as float32; a bad id raises ``status`` (int32[1])."""
     _need_cuda(table, ids, out, status)
     T, width = out.shape
     assert out.dtype == torch.float32 and ids.dtype == torch.int32 and out.is_contiguous()
     assert table.is_contiguous() and table.shape[1] == width
     _check(_lib("basic.cu").ub_embed(_ptr(table), _code(table), _ptr(ids), _ptr(out), T, width,
-                                     table.shape[0], _ptr(status), _stream()), "embed")
+                                     table.shape[0], _ptr(status), float(scale), _stream()), "embed")
 
 
 def embed_pairs(table, pairs, ids, batch, last, out, status, scale, buckets, mul_prev, mul_cur):
@@ -332,14 +333,16 @@ def rmsnorm_add(y, weight, x, eps, h=None, clear_y=False):
                                            n, width, float(eps), 1 if clear_y else 0, _stream()), "rmsnorm_add")
 
 
-def glu_clamped(gate_up, out, limit, alpha, shift):
+def glu_clamped(gate_up, out, limit, alpha, shift, row_gate=None):
     """out = g' * sigmoid(alpha g') * (u' + shift) with g' = min(g, limit), u' = clamp(u, -limit, limit);
-    gate_up [T, 2F] holds g and u side by side."""
-    _need_cuda(gate_up, out)
+    gate_up [T, 2F] holds g and u side by side.  ``row_gate`` float32 [T] (any stride): a row times its sigmoid."""
+    _need_cuda(gate_up, out, row_gate)
+    assert row_gate is None or (row_gate.dtype == torch.float32 and row_gate.dim() == 1 and row_gate.numel() == out.shape[0])
     T, F = out.shape
     assert gate_up.shape == (T, 2 * F) and gate_up.is_contiguous() and out.is_contiguous()
     _check(_lib("basic.cu").ub_glu_clamped(_ptr(gate_up), _code(gate_up), _ptr(out), _code(out), T, F, float(limit),
-                                           float(alpha), float(shift), _stream()), "glu_clamped")
+                                           float(alpha), float(shift), _ptr(row_gate),
+                                           row_gate.stride(0) if row_gate is not None else 0, _stream()), "glu_clamped")
 
 
 def head_gate(o, gate, n_heads, head_dim):
@@ -540,10 +543,11 @@ def gemm_batched(a, w, out):
                                                      _stream()), "gemm_batched")
 
 
-def gemm_grouped(a, w, out, tiles, n_tiles, src_rows, max_tiles, epilogue=EPI_STORE, w2=None):
+def gemm_grouped(a, w, out, tiles, n_tiles, src_rows, max_tiles, epilogue=EPI_STORE, w2=None, gate=None):
     """Sorted rows against the matrix their tile names: out[p, :] = a[src_rows[p] (or p), :] @ w[e].T; w [E, N, K]
     contiguous; EPI_SWIGLU: out = silu(a w[e]^T) * (a w2[e]^T), w2 a view with w's strides.  ``tiles`` int32
-    [max_tiles, 4] (matrix, first row, rows, -) and ``n_tiles`` int32 [1] on the device (csrc/routed.cu makes them)."""
+    [max_tiles, 4] (matrix, first row, rows, -) and ``n_tiles`` int32 [1] on the device (csrc/routed.cu makes them).
+    ``gate`` = (limit, alpha, shift): the constants of the gate product (see ``glu_clamped``)."""
     _need_cuda(a, w, out, tiles, n_tiles, src_rows)
     E, N, K = w.shape
     assert w.stride(2) == 1 and w.stride(1) >= K and a.stride(1) == 1 and out.stride(1) == 1 and out.shape[1] == N and a.shape[1] == K
@@ -552,7 +556,8 @@ def gemm_grouped(a, w, out, tiles, n_tiles, src_rows, max_tiles, epilogue=EPI_ST
         assert w2.shape == w.shape and w2.stride() == w.stride() and w2.dtype == w.dtype
     _check(_lib("gemm_simt.cu").ub_gemm_simt_grouped(_ptr(a), _code(a), _ptr(w), _ptr(w2), _code(w), _ptr(out), _code(out), N, K,
                                                      a.stride(0), w.stride(1), out.stride(0), w.stride(0), _ptr(tiles),
-                                                     _ptr(n_tiles), _ptr(src_rows), int(max_tiles), epilogue, _stream()),
+                                                     _ptr(n_tiles), _ptr(src_rows), int(max_tiles), epilogue,
+                                                     (c_float * 3)(*gate[:3]) if gate is not None else None, _stream()),
            "gemm_grouped")
 
 
@@ -561,32 +566,39 @@ def gemm_grouped(a, w, out, tiles, n_tiles, src_rows, max_tiles, epilogue=EPI_ST
 ROUTE_TILE = 64          # sorted rows a tile of the grouped products
 
 
-ROUTE_SIGMOID, ROUTE_GROUP_TOP2, ROUTE_NORMALISE = 1, 2, 4      # bits of a router's ``mode`` (csrc/routed.cu)
+ROUTE_SIGMOID, ROUTE_GROUP_TOP2, ROUTE_NORMALISE, ROUTE_LOGITS = 1, 2, 4, 8      # bits of a router's ``mode`` (csrc/routed.cu)
 
 
-def route(z, correction, n_experts, top, n_groups, keep, idx, wts, counts, mode=0, wscale=1.0):
+def _router_columns(z, extra):
+    """The router's outputs among the columns of z: all of them, or all but one where ``extra`` (float32 [T]) takes the last."""
+    assert extra is None or (extra.dtype == torch.float32 and extra.is_contiguous() and extra.numel() == z.shape[-2])
+    return z.shape[-1] - (1 if extra is not None else 0)
+
+
+def route(z, correction, n_experts, top, n_groups, keep, idx, wts, counts, mode=0, wscale=1.0, extra=None):
     """z float32 [T, outputs] router logits (or [parts, T, outputs], summed in that order) -> idx int32 [T, top], wts
-    float32 [T, top]; counts int32 [n_experts] += rows.  ``mode``: ROUTE_* bits; ``wscale`` multiplies the weights."""
-    _need_cuda(z, correction, idx, wts, counts)
+    float32 [T, top]; counts int32 [n_experts] += rows.  ``mode``: ROUTE_* bits; ``wscale`` multiplies the weights.  ``extra``
+    float32 [T]: z has one column behind the outputs, whose sums over the parts go there."""
+    _need_cuda(z, correction, idx, wts, counts, extra)
     T, ldz, n_parts, part_stride = _parts_of(z)
-    n_out = z.shape[-1]
+    n_out = _router_columns(z, extra)
     assert z.dtype == torch.float32 and z.stride(-1) == 1 and idx.dtype == torch.int32 and wts.dtype == torch.float32
     assert idx.is_contiguous() and wts.is_contiguous() and idx.shape == wts.shape == (T, top) and counts.dtype == torch.int32
     assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == n_out)
     _check(_lib("routed.cu").ub_route(_ptr(z), ldz, n_parts, part_stride, _ptr(correction), T, n_out, n_experts, top, n_groups, keep,
-                                      _ptr(idx), _ptr(wts), _ptr(counts), int(mode), float(wscale), _stream()), "route")
+                                      _ptr(idx), _ptr(wts), _ptr(counts), int(mode), float(wscale), _ptr(extra), _stream()), "route")
 
 
 ROUTE_SMALL_TOKENS = 16      # steps of at most this many tokens (a warp each): route, plan and scatter as one launch (csrc/routed.cu)
 
 
 def route_small(z, correction, n_experts, top, n_groups, keep, idx, wts, tiles, n_tiles, row_pos, src_rows, tile, mode=0,
-                wscale=1.0):
+                wscale=1.0, extra=None):
     """``route``, ``route_plan`` and ``route_scatter`` of a step of at most ROUTE_SMALL_TOKENS tokens in one launch of one
     block; the counters of the separate kernels are not used."""
-    _need_cuda(z, correction, idx, wts, tiles, n_tiles, row_pos, src_rows)
+    _need_cuda(z, correction, idx, wts, tiles, n_tiles, row_pos, src_rows, extra)
     T, ldz, n_parts, part_stride = _parts_of(z)
-    n_out = z.shape[-1]
+    n_out = _router_columns(z, extra)
     assert T <= ROUTE_SMALL_TOKENS and z.dtype == torch.float32 and z.stride(-1) == 1
     assert idx.dtype == torch.int32 and wts.dtype == torch.float32 and idx.is_contiguous() and wts.is_contiguous()
     assert idx.shape == wts.shape == (T, top) and row_pos.dtype == src_rows.dtype == torch.int32
@@ -595,7 +607,7 @@ def route_small(z, correction, n_experts, top, n_groups, keep, idx, wts, tiles, 
     assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == n_out)
     _check(_lib("routed.cu").ub_route_small(_ptr(z), ldz, n_parts, part_stride, _ptr(correction), T, n_out, n_experts, top,
                                             n_groups, keep, _ptr(idx), _ptr(wts), _ptr(tiles), _ptr(n_tiles), _ptr(row_pos),
-                                            _ptr(src_rows), tile, int(mode), float(wscale), _stream()), "route_small")
+                                            _ptr(src_rows), tile, int(mode), float(wscale), _ptr(extra), _stream()), "route_small")
 
 
 def route_plan(counts, cursor, seg_start, tiles, n_tiles, n_experts, tile=ROUTE_TILE):
@@ -636,23 +648,43 @@ def route_combine(y, h, row_pos, wts, residual):
 
 # ---------------------------------------------------------------------------------------
 # latent attention (csrc/latent.cu)
-def latent_place(x, q_off, c_off, q_plain, q_lat, c_weight, cos, sin, rotary_dim, tok_pos, tok_seq, k_cache, table, ring, page,
-                 n_heads, dim, rot, rank, eps):
-    """From projection rows x ([T, N] or [parts, T, N], summed): the heads' unrotated query parts into q_plain
-    [T, heads, dim], their rotated parts into q_lat[:, :, rank:] ([T, heads, rank + rot]), and the position's cache row
-    [normed latent | rotated key part]."""
-    _need_cuda(x, q_plain, q_lat, k_cache, table)
+def latent_place(x, k_cache=None, table=None, ring=0, page=1, tok_pos=None, tok_seq=None, c_off=None, c_weight=None, rank=0, rot=0,
+                 cos=None, sin=None, rotary_dim=0, eps=0.0, q_off=None, q_plain=None, q_lat=None, n_heads=0, dim=0,
+                 dq_off=None, dq_weight=None, dq_out=None, g_off=None, gate_out=None):
+    """From projection rows x ([T, N] or [parts, T, N], summed), whichever of these are asked for:
+      c_off    the position's cache row [normed latent | rotated key part]
+      q_off    the heads' unrotated query parts into q_plain [T, heads, dim] and their rotated parts into q_lat[:, :, rank:]
+               ([T, heads, rank + rot])
+      dq_off   the queries' latent, RMS-normed with ``dq_weight``, into dq_out [T, q_rank]
+      g_off    gate columns as they are into gate_out (float32 [T, columns])"""
+    _need_cuda(x, q_plain, q_lat, k_cache, table, dq_out, gate_out)
     T, ldx, n_parts, part_stride = _parts_of(x)
-    assert q_plain.is_contiguous() and q_lat.is_contiguous() and q_plain.dtype == q_lat.dtype
-    assert q_plain.shape == (T, n_heads, dim) and q_lat.shape == (T, n_heads, rank + rot)
-    assert c_weight.dtype == torch.float32 and c_weight.is_contiguous() and c_weight.numel() == rank
-    assert table.dtype == torch.int32 and table.dim() == 2 and table.is_contiguous()
+    act = [t for t in (q_plain, q_lat, dq_out) if t is not None]
+    for t in act:
+        assert t.is_contiguous() and t.dtype == act[0].dtype
+    if q_off is not None:
+        assert q_plain.shape == (T, n_heads, dim) and q_lat.shape == (T, n_heads, rank + rot)
+    if c_off is not None:
+        assert c_weight.dtype == torch.float32 and c_weight.is_contiguous() and c_weight.numel() == rank
+        assert table.dtype == torch.int32 and table.dim() == 2 and table.is_contiguous()
+    if dq_off is not None:
+        assert dq_weight.dtype == torch.float32 and dq_weight.is_contiguous() and dq_out.shape == (T, dq_weight.numel())
+    if g_off is not None:
+        assert gate_out.dtype == torch.float32 and gate_out.is_contiguous() and gate_out.shape[0] == T
     if cos is not None:
         assert cos.dtype == torch.float32 and cos.is_contiguous() and cos.shape[1] == rotary_dim // 2 and sin.shape == cos.shape
+
+    def at(off):
+        return -1 if off is None else int(off)
+    code = _code(k_cache if k_cache is not None else act[0])          # the cache has the activations' type
+    assert all(_code(t) == code for t in act)
     _check(_lib("latent.cu").ub_latent_place(
-        _ptr(x), _code(x), ldx, n_parts, part_stride, int(q_off), int(c_off), _ptr(q_plain), _ptr(q_lat), _code(q_lat),
-        _ptr(c_weight), _ptr(cos), _ptr(sin), int(rotary_dim or 0), _ptr(tok_pos), _ptr(tok_seq), _ptr(k_cache), _code(k_cache),
-        _ptr(table), table.shape[1], ring, page, T, n_heads, dim, rot, rank, float(eps), _stream()), "latent_place")
+        _ptr(x), _code(x), ldx, n_parts, part_stride,
+        at(dq_off), _ptr(dq_weight), dq_weight.numel() if dq_off is not None else 0, _ptr(dq_out),
+        at(q_off), _ptr(q_plain), _ptr(q_lat), code, at(c_off), _ptr(c_weight), _ptr(cos), _ptr(sin), int(rotary_dim or 0),
+        _ptr(k_cache), code, at(g_off), gate_out.shape[1] if g_off is not None else 0, _ptr(gate_out), _ptr(tok_pos), _ptr(tok_seq),
+        _ptr(table), table.shape[1] if table is not None else 0, ring, page, T, n_heads, dim, rot, rank, float(eps), _stream()),
+        "latent_place")
 
 
 # ---------------------------------------------------------------------------------------
@@ -802,31 +834,49 @@ def delta_finish(o, gate_pre, weight, out, H, E, eps, silu_gate=False):
 # ---------------------------------------------------------------------------------------
 # ---------------------------------------------------------------------------------------
 # row-wise kernels of a stream with scaled sublayers and input convolutions (csrc/rowwise.cu)
-def layernorm(x, weight, out, eps, rows=None):
-    """out = (x - mean) / sqrt(var + eps) * weight row by row (no bias); x float32 [T, width]; ``rows`` int32: only these."""
-    _need_cuda(x, weight, out, rows)
+def layernorm(x, weight, out, eps, rows=None, bias=None):
+    """out = (x - mean) / sqrt(var + eps) * weight (+ bias) row by row; x float32 [T, width]; ``rows`` int32: only these."""
+    _need_cuda(x, weight, out, rows, bias)
     width = x.shape[1]
     assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[1] == width
     assert weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == width
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == width)
     n = x.shape[0] if rows is None else rows.numel()
     assert out.shape[0] == n
-    _check(_lib("rowwise.cu").ub_layernorm(_ptr(x), _ptr(weight), _ptr(out), _code(out), _ptr(rows), n, width, float(eps),
+    _check(_lib("rowwise.cu").ub_layernorm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(out), _code(out), _ptr(rows), n, width, float(eps),
                                            _stream()), "layernorm")
 
 
 NEXT_NONE, NEXT_PLAIN, NEXT_RMS, NEXT_LAYER = 0, 1, 2, 3
 
 
-def scale_add_norm(y, scale, x, mode=NEXT_NONE, norm_weight=None, eps=0.0, out=None, clear_y=True):
-    """x += scale * y (``scale`` float32 [width] or None for 1), y cleared; ``out`` receives what the next sublayer reads:
-    the new x as it is (NEXT_PLAIN), its RMS norm (NEXT_RMS) or its layer norm (NEXT_LAYER) times ``norm_weight``."""
-    _need_cuda(y, scale, x, norm_weight, out)
+def norm_join(y, x, mult, after, mode=NEXT_NONE, then=None, out=None, clear_y=True):
+    """x += mult * norm(y), y cleared; ``after`` = (NEXT_RMS or NEXT_LAYER, weight, bias or None, eps) is that norm.  ``out`` receives
+    what the next sublayer reads: the new x as it is (NEXT_PLAIN) or its norm, ``then`` = (weight, bias or None, eps)."""
+    kind, aw, ab, a_eps = after
+    nw, nb, n_eps = then if then is not None else (None, None, 0.0)
+    _need_cuda(y, x, aw, ab, nw, nb, out)
     T, width = x.shape
     assert x.dtype == y.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and y.shape == x.shape
-    for v in (scale, norm_weight):
+    assert kind in (NEXT_RMS, NEXT_LAYER)
+    for v in (aw, ab, nw, nb):
         assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == width)
     assert out is None or (out.is_contiguous() and tuple(out.shape) == (T, width))
-    _check(_lib("rowwise.cu").ub_scale_add_norm(_ptr(y), _ptr(scale), _ptr(x), int(mode), _ptr(norm_weight), float(eps), _ptr(out),
+    _check(_lib("rowwise.cu").ub_norm_join(_ptr(y), _ptr(x), float(mult), _ptr(aw), _ptr(ab), float(a_eps), 1 if kind == NEXT_LAYER else 0,
+                                           int(mode), _ptr(nw), _ptr(nb), float(n_eps), _ptr(out),
+                                           _code(out) if out is not None else F32, T, width, 1 if clear_y else 0, _stream()), "norm_join")
+
+
+def scale_add_norm(y, scale, x, mode=NEXT_NONE, norm_weight=None, eps=0.0, out=None, clear_y=True, norm_bias=None):
+    """x += scale * y (``scale`` float32 [width] or None for 1), y cleared; ``out`` receives what the next sublayer reads:
+    the new x as it is (NEXT_PLAIN), its RMS norm (NEXT_RMS) or its layer norm (NEXT_LAYER) times ``norm_weight`` (+ ``norm_bias``)."""
+    _need_cuda(y, scale, x, norm_weight, out, norm_bias)
+    T, width = x.shape
+    assert x.dtype == y.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and y.shape == x.shape
+    for v in (scale, norm_weight, norm_bias):
+        assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == width)
+    assert out is None or (out.is_contiguous() and tuple(out.shape) == (T, width))
+    _check(_lib("rowwise.cu").ub_scale_add_norm(_ptr(y), _ptr(scale), _ptr(x), int(mode), _ptr(norm_weight), _ptr(norm_bias), float(eps), _ptr(out),
                                                 _code(out) if out is not None else F32, T, width, 1 if clear_y else 0, _stream()),
            "scale_add_norm")
 

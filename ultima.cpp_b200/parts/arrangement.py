@@ -89,6 +89,73 @@ class NormAfterMixerOnly(_NormAfter):
         pass
 
 
+class _NormBoth(Arrangement):
+    """x += mult * norm_after(mixer(norm(x))); x += mult * norm_after(feed_forward(norm(x))): a norm on what a sublayer reads and
+    one on what it puts out (norms of kind "rms" or "layer").  A sublayer adds its output into a cleared float32 buffer y; ONE
+    kernel a sublayer norms y, folds it into x, clears y and writes what the next sublayer reads: the feed-forward's norm of
+    the new x behind the mixer, the next layer's first norm behind the feed-forward (``Runtime.next_layer``, where that
+    layer has this arrangement too).  Both buffers are kept from layer to layer of a pass."""
+
+    def __init__(self, mult: float = 1.0):
+        self.mult = float(mult)
+
+    def kernel_needs(self, run_dtype):
+        return [("rowwise.cu", ())]
+
+    def _buffers(self, x, rt):
+        key = (rt.pass_id, x.data_ptr(), tuple(x.shape))
+        carry = getattr(rt, "_norm_both_carry", None)
+        if carry is None or carry[0] != key:
+            y = rt.arena.alloc(tuple(x.shape), x.dtype)
+            y.zero_()
+            carry = rt._norm_both_carry = [key, rt.arena.alloc(tuple(x.shape), rt.dtype), y, None]     # (last: the layer h was made for)
+        return carry
+
+    def _join(self, y, x, h, after, then, rt):
+        """``then``: the norm whose output of the new x goes into h, or None.  True if h was written."""
+        kinds = {"rms": ops.NEXT_RMS, "layer": ops.NEXT_LAYER}
+        if after.kind not in kinds:
+            raise ValueError(f"norm_both: a norm of kind '{after.kind}' behind a sublayer is not one the joining kernel takes")
+        mode = kinds.get(then.kind) if then is not None else None
+        rt.launches += 1
+        ops.norm_join(y, x, self.mult, (kinds[after.kind], after.weight, getattr(after, "bias", None), after.eps),
+                      mode or ops.NEXT_NONE, (then.weight, getattr(then, "bias", None), then.eps) if mode else None, h if mode else None)
+        return mode is not None
+
+    def run(self, layer, x, batch, cache, rt):
+        carry = self._buffers(x, rt)
+        _, h, y, made_for = carry
+        mark = rt.arena.mark()
+        if made_for is not layer:
+            h = layer.mixer_norm.forward(x, rt)
+        ff = getattr(layer, "feed_forward", None)
+        nxt = getattr(rt, "next_layer", None)
+        if nxt is not None and not isinstance(nxt.arrangement, _NormBoth):
+            nxt = None
+        layer.mixer.forward(h, y, batch, cache, rt)
+        rt.arena.reset(mark)
+        h, after = carry[1], layer.mixer_norm_after
+        if ff is not None:
+            if not self._join(y, x, h, after, layer.feed_forward_norm, rt):
+                h = layer.feed_forward_norm.forward(x, rt)
+            ff.forward(h, y, batch, rt)
+            rt.arena.reset(mark)
+            h, after = carry[1], layer.feed_forward_norm_after
+        carry[3] = nxt if self._join(y, x, h, after, nxt.mixer_norm if nxt is not None else None, rt) else None
+
+
+@register_part("arrangement", "norm_both")
+class NormBoth(_NormBoth):
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_norm_after": "norm", "feed_forward_norm": "norm",
+             "feed_forward": "feed_forward", "feed_forward_norm_after": "norm"}
+
+
+@register_part("arrangement", "norm_both_mixer_only")
+class NormBothMixerOnly(_NormBoth):
+    """The same layer without a feed-forward."""
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_norm_after": "norm"}
+
+
 @register_part("residual_gate", "sigmoid_linear")
 class SigmoidLinearGate(ResidualGate):
     """x += sigmoid(W h + b) * y, element by element: a square projection of the sublayer's own input opens

@@ -361,7 +361,8 @@ class ModelSpec:
     def kernel_needs(self, run_dtype) -> list:
         """Every library the model's parts ask for (see ``Part.kernel_needs``), once each."""
         out = []
-        for _, family, ps in self.parts_with_names():
+        held = [("arrangement", L.arrangement) for L in self.layers] + [(family, ps) for _, family, ps in self.parts_with_names()]
+        for family, ps in held:
             for t in build_part(family, ps).kernel_needs(run_dtype):
                 t = (t[0], tuple(t[1]))
                 if t not in out:

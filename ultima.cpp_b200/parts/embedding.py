@@ -10,17 +10,17 @@ from .base import Part, StateNeed, register_part
 
 @register_part("embedding", "token_table")
 class TokenTable(Part):
-    """x_t = E[id_t, :], no scaling (reference: src/model/qwen_model.cpp:145-157).  A token id
+    """x_t = scale * E[id_t, :] (reference, without a scale: src/model/qwen_model.cpp:145-157).  A token id
     outside the vocabulary is refused on the host before the launch; the kernel checks again
     and raises a flag."""
 
-    def __init__(self, vocab_size: int, width: int, norm: str | None = None, eps: float = 0.0):
+    def __init__(self, vocab_size: int, width: int, norm: str | None = None, eps: float = 0.0, scale: float = 1.0):
         """``norm``: "layer" or "rms": the gathered rows pass a norm with a weight of its own (tensor ``norm.weight``) and
         ``eps`` before they enter the stream (float32 in and out)."""
         self.vocab_size, self.width = int(vocab_size), int(width)
         if norm not in (None, "layer", "rms"):
             raise ValueError("token_table: norm is 'layer', 'rms' or None")
-        self.norm, self.eps = norm, float(eps)
+        self.norm, self.eps, self.scale = norm, float(eps), float(scale)
         self.table = self.norm_w = None
 
     def weight_specs(self):
@@ -41,7 +41,7 @@ class TokenTable(Part):
     def forward(self, ids, rt):
         x = rt.arena.alloc((ids.numel(), self.width), torch.float32)
         rt.launches += 1
-        ops.embed(self.table, ids, x, self.status)
+        ops.embed(self.table, ids, x, self.status, self.scale)
         if self.norm:
             out = rt.arena.alloc((ids.numel(), self.width), torch.float32)
             rt.launches += 1

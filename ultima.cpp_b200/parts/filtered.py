@@ -17,16 +17,16 @@ from .base import Arrangement, InputFilter, ResidualGate, StateNeed, Tail, regis
 
 
 def _next_mode(then):
-    """How the joining kernel writes what the next reader wants: (mode, weight, eps), or None if it cannot."""
+    """How the joining kernel writes what the next reader wants: (mode, weight, bias, eps), or None if it cannot."""
     if then is None:
-        return ops.NEXT_NONE, None, 0.0
+        return ops.NEXT_NONE, None, None, 0.0
     if then == "plain":
-        return ops.NEXT_PLAIN, None, 0.0
+        return ops.NEXT_PLAIN, None, None, 0.0
     kind = getattr(then, "kind", None)
     if kind == "layer":
-        return ops.NEXT_LAYER, then.weight, then.eps
+        return ops.NEXT_LAYER, then.weight, then.bias, then.eps
     if kind == "rms":
-        return ops.NEXT_RMS, then.weight, then.eps
+        return ops.NEXT_RMS, then.weight, None, then.eps
     return None
 
 
@@ -46,12 +46,12 @@ class _ChannelGate(ResidualGate):
         if how is None:
             ops.scale_add_norm(y, self.scale, x)
             return then.forward(x, rt)
-        mode, w, eps = how
+        mode, w, b, eps = how
         if mode == ops.NEXT_PLAIN and rt.dtype == x.dtype:
             ops.scale_add_norm(y, self.scale, x)
             return x                                   # a 32-bit run reads the stream itself
         out = rt.arena.alloc(tuple(x.shape), rt.dtype) if mode != ops.NEXT_NONE else None
-        ops.scale_add_norm(y, self.scale, x, mode, w, eps, out)
+        ops.scale_add_norm(y, self.scale, x, mode, w, eps, out, norm_bias=b)
         return out
 
 

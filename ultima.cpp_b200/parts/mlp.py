@@ -87,18 +87,20 @@ class GatedClamped(FeedForward):
         else:
             self.wgu = torch.cat([g, u], dim=0).contiguous()
 
-    def forward(self, h, residual, batch, rt):
+    def forward(self, h, residual, batch, rt, row_gate=None):
+        """``row_gate`` (float32 [T], any stride): a token's result times the sigmoid of its number (on the gate product)."""
         T = h.shape[0]
         if self.interleaved:
             a = rt.arena.alloc((T, self.inner), rt.dtype)
-            rt.matmul(h, self.wgu, a, ops.EPI_SWIGLU_IL, gate=(self.limit, self.alpha, self.shift))
+            rt.matmul(h, self.wgu, a, ops.EPI_SWIGLU_IL, gate=(self.limit, self.alpha, self.shift),
+                      mul=None if row_gate is None else (row_gate, 0))
             rt.matmul(a, self.wd, residual, ops.EPI_ADD)
             return
         gu = rt.arena.alloc((T, 2 * self.inner), torch.float32)
         rt.matmul(h, self.wgu, gu)
         a = rt.arena.alloc((T, self.inner), rt.dtype)
         rt.launches += 1
-        ops.glu_clamped(gu, a, self.limit, self.alpha, self.shift)
+        ops.glu_clamped(gu, a, self.limit, self.alpha, self.shift, row_gate)
         rt.matmul(a, self.wd, residual, ops.EPI_ADD)
 
 

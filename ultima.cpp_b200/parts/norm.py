@@ -38,16 +38,19 @@ class RMSNorm(Norm):
 
 @register_part("norm", "layer")
 class LayerNorm(Norm):
-    """y = (x - mean) / sqrt(var + eps) * w, the variance being the mean of the squared deviations; a weight and no
-    bias.  ``scale``: a constant folded into the weight (a model that multiplies its logits by a constant puts it on
+    """y = (x - mean) / sqrt(var + eps) * w (+ b with ``with_bias``), the variance being the mean of the squared deviations.
+    ``scale``: a constant folded into weight and bias (a model that multiplies its logits by a constant puts it on
     the final norm).  Input is the float32 residual stream, sums are float32, the output has the activation type."""
 
-    def __init__(self, width: int, eps: float, scale: float = 1.0):
-        self.width, self.eps, self.scale = int(width), float(eps), float(scale)
-        self.weight = None
+    def __init__(self, width: int, eps: float, scale: float = 1.0, with_bias: bool = False):
+        self.width, self.eps, self.scale, self.with_bias = int(width), float(eps), float(scale), bool(with_bias)
+        self.weight = self.bias = None
 
     def weight_specs(self):
-        return [WeightSpec("weight", (self.width,), "vector", ("one_plus_normal", 0.05))]
+        s = [WeightSpec("weight", (self.width,), "vector", ("one_plus_normal", 0.05))]
+        if self.with_bias:
+            s.append(WeightSpec("bias", (self.width,), "vector", ("normal", 0.1)))
+        return s
 
     def kernel_needs(self, run_dtype):
         return [("rowwise.cu", ())]
@@ -55,10 +58,13 @@ class LayerNorm(Norm):
     def bind(self, tensors, rt):
         w = tensors["weight"].float()
         self.weight = (w * self.scale if self.scale != 1.0 else w).contiguous()
+        if self.with_bias:
+            b = tensors["bias"].float()
+            self.bias = (b * self.scale if self.scale != 1.0 else b).contiguous()
 
     def forward(self, x, rt, rows=None):
         n = x.shape[0] if rows is None else rows.numel()
         out = rt.arena.alloc((n, self.width), rt.dtype)
         rt.launches += 1
-        ops.layernorm(x, self.weight, out, self.eps, rows)
+        ops.layernorm(x, self.weight, out, self.eps, rows, bias=self.bias)
         return out

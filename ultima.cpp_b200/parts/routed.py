@@ -39,7 +39,13 @@ class RoutedExperts(FeedForward):
       group_score="top2_sum" a group's score is the sum of its two largest choice scores instead of the largest
       normalise=True         the chosen outputs' weights are divided by their sum (+ 1e-20)
       weight_scale           a constant on the weights (behind the normalisation)
+      score="logits"         s = z itself; the chosen outputs' weights are the softmax over the chosen logits only
       expert="relu_squared"  an expert (and the shared one) is down(max(up h, 0)^2): no gate matrix
+      expert="gated_clamped" an expert is down(g' sigmoid(alpha g') (u' + shift)) with g' = min(gate h, limit) and u' =
+                             clamp(up h, -limit, limit); ``clamp`` = (limit, alpha, shift), and ``shared_limit`` the shared
+                             expert's limit where it is not the others'
+      shared_gate=True       the shared expert's result is multiplied by the sigmoid of one number a token, w . h (tensor
+                             ``shared.out_gate.weight`` [1, width]; one more row of the router's product); gated experts only
 
     On the GPU: the router's product with float32 sums (CUDA cores and float32 weights; in a bfloat16 run the stored
     bfloat16 weights on the tensor cores, whose products of two bfloat16 numbers are exact); one kernel picks and counts, one lays
@@ -55,7 +61,8 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, width: int, inner: int, n_experts: int, top: int, n_identity: int = 0, groups: tuple | None = None,
                  shared_inner: int | None = None, correction: bool = True, score: str = "softmax", group_score: str = "max",
-                 normalise: bool = False, weight_scale: float = 1.0, expert: str = "gated_silu"):
+                 normalise: bool = False, weight_scale: float = 1.0, expert: str = "gated_silu", clamp: tuple | None = None,
+                 shared_limit: float | None = None, shared_gate: bool = False):
         self.width, self.inner, self.ne, self.top = int(width), int(inner), int(n_experts), int(top)
         self.ni = int(n_identity or 0)
         self.n_out = self.ne + self.ni
@@ -65,16 +72,29 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: top must not exceed the router's outputs, which divide into equal groups")
         if self.n_out > 1024 or self.ne < 1:
             raise ValueError("routed_experts: the router kernel takes up to 1,024 outputs, at least one of them an expert")
-        if score not in ("softmax", "sigmoid") or group_score not in ("max", "top2_sum") or expert not in ("gated_silu", "relu_squared"):
-            raise ValueError("routed_experts: score is 'softmax' or 'sigmoid', group_score 'max' or 'top2_sum', expert "
-                             "'gated_silu' or 'relu_squared'")
-        self.mode = ((ops.ROUTE_SIGMOID if score == "sigmoid" else 0) | (ops.ROUTE_GROUP_TOP2 if group_score == "top2_sum" else 0)
+        if (score not in ("softmax", "sigmoid", "logits") or group_score not in ("max", "top2_sum")
+                or expert not in ("gated_silu", "relu_squared", "gated_clamped")):
+            raise ValueError("routed_experts: score is 'softmax', 'sigmoid' or 'logits', group_score 'max' or 'top2_sum', expert "
+                             "'gated_silu', 'relu_squared' or 'gated_clamped'")
+        self.mode = ({"softmax": 0, "sigmoid": ops.ROUTE_SIGMOID, "logits": ops.ROUTE_LOGITS}[score] | (ops.ROUTE_GROUP_TOP2 if group_score == "top2_sum" else 0)
                      | (ops.ROUTE_NORMALISE if normalise else 0))
-        self.weight_scale, self.gated = float(weight_scale), expert == "gated_silu"
+        self.weight_scale, self.gated = float(weight_scale), expert != "relu_squared"
+        if (expert == "gated_clamped") != (clamp is not None):
+            raise ValueError("routed_experts: clamp = (limit, alpha, shift) goes with 'gated_clamped' experts")
+        self.clamp = tuple(float(v) for v in clamp) if clamp is not None else None
+        self.shared_gate = bool(shared_gate) and bool(shared_inner)
+        if self.shared_gate and self.clamp is None:
+            raise ValueError("routed_experts: a gate on the shared expert goes with 'gated_clamped' experts")
         if not self.gated and self.ni:
             raise ValueError("routed_experts: identity experts go with gated experts")
-        shared = part("gated_silu", width=self.width, inner=int(shared_inner or 0)) if self.gated else \
-            part("plain_mlp", width=self.width, inner=int(shared_inner or 0), activation="relu_squared")
+        if self.clamp is not None:
+            limit, alpha, shift = self.clamp
+            shared = part("gated_clamped", width=self.width, inner=int(shared_inner or 0), alpha=alpha, shift=shift,
+                          limit=limit if shared_limit is None else float(shared_limit))
+        elif self.gated:
+            shared = part("gated_silu", width=self.width, inner=int(shared_inner or 0))
+        else:
+            shared = part("plain_mlp", width=self.width, inner=int(shared_inner or 0), activation="relu_squared")
         self.shared = build_part("feed_forward", shared) if shared_inner else None
 
     def weight_specs(self):
@@ -89,6 +109,8 @@ class RoutedExperts(FeedForward):
                   W(f"experts.{e}.down_proj.weight", (self.width, self.inner))]
         if self.shared is not None:
             s += [W("shared." + w.name, w.shape, w.kind, w.init) for w in self.shared.weight_specs()]
+            if self.shared_gate:
+                s.append(W("shared.out_gate.weight", (1, self.width), "matrix", ("normal", 0.3)))
         return s
 
     def kernel_needs(self, run_dtype):
@@ -104,6 +126,8 @@ class RoutedExperts(FeedForward):
         # products, so that pair may go to the tensor cores, which add them up in float32; anything else runs on the
         # CUDA cores with float32 weights
         wr = tensors["router.weight"]
+        if self.shared_gate:                                         # the shared expert's gate: one more row of the same product
+            wr = torch.cat([wr, tensors["shared.out_gate.weight"].to(wr.dtype)], dim=0)
         self.w_router = wr.contiguous() if (wr.dtype == torch.bfloat16 and rt.dtype == torch.bfloat16 and self.width % 8 == 0) \
             else wr.float().contiguous()
         self.corr = tensors["correction"].float().contiguous() if self.correction else None
@@ -129,8 +153,15 @@ class RoutedExperts(FeedForward):
         i32, f32 = torch.int32, torch.float32
         z = rt.matmul_parts(h, self.w_router)          # few tokens: K in slices, summed by the routing kernel
         if z is None:
-            z = rt.arena.alloc((T, self.n_out), f32)
+            z = rt.arena.alloc((T, self.w_router.shape[0]), f32)
             rt.matmul(h, self.w_router, z)
+        # the shared expert's gate: the router product's last column, summed over K slices by the routing kernel where there are any
+        shared_gate = extra = None
+        if self.shared_gate:
+            if z.dim() == 3:
+                shared_gate = extra = rt.arena.alloc((T,), f32)
+            else:
+                shared_gate, z = z[:, self.n_out], z[:, :self.n_out]
         idx = rt.arena.alloc((T, top), i32)
         wts = rt.arena.alloc((T, top), f32)
         row_pos = rt.arena.alloc((T, top), i32)
@@ -156,10 +187,11 @@ class RoutedExperts(FeedForward):
         if T <= ops.ROUTE_SMALL_TOKENS and self._small_fits:
             rt.launches += 1                  # few tokens: the three steps as one launch of one block
             ops.route_small(z, self.corr, ne, top, self.groups[0], self.groups[1], idx, wts, tiles, n_tiles, row_pos, src_rows, tile,
-                            mode=self.mode, wscale=self.weight_scale)
+                            mode=self.mode, wscale=self.weight_scale, extra=extra)
         else:
             rt.launches += 3
-            ops.route(z, self.corr, ne, top, self.groups[0], self.groups[1], idx, wts, counts, mode=self.mode, wscale=self.weight_scale)
+            ops.route(z, self.corr, ne, top, self.groups[0], self.groups[1], idx, wts, counts, mode=self.mode, wscale=self.weight_scale,
+                      extra=extra)
             ops.route_plan(counts, cursor, seg_start, tiles, n_tiles, ne, tile)
             ops.route_scatter(idx, seg_start, cursor, row_pos, src_rows, ne)
         plan = RoutePlan(tiles, n_tiles, src_rows, max_tiles, T * top, tile=tile)
@@ -168,12 +200,15 @@ class RoutedExperts(FeedForward):
             rt.launches += 1
             ops.route_gather(h, row_pos, rows)
             plan.gather = False
-            rt.matmul_grouped(rows, first[0], first[1], plan, first[2], w2=first[3], unary=unary)
+            rt.matmul_grouped(rows, first[0], first[1], plan, first[2], w2=first[3], unary=unary, gate=self.clamp)
         else:
-            rt.matmul_grouped(h, first[0], first[1], plan, first[2], w2=first[3], unary=unary)
+            rt.matmul_grouped(h, first[0], first[1], plan, first[2], w2=first[3], unary=unary, gate=self.clamp)
         plan.gather = False
         rt.matmul_grouped(act, self.w_down, y, plan)
         rt.launches += 1
         ops.route_combine(y, h, row_pos, wts, residual)
         if self.shared is not None:
-            self.shared.forward(h, residual, batch, rt)
+            if self.shared_gate:
+                self.shared.forward(h, residual, batch, rt, row_gate=shared_gate)
+            else:
+                self.shared.forward(h, residual, batch, rt)
