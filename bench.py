@@ -528,6 +528,28 @@ def bizepel_config(z):
             "token_side": {"dim": 256}, "logit_scale": 1.0, "layers": layers}
 
 
+def bozavik_config(z):
+    """Layers in pairs: latent attention with a rotated part and a gate a head, latent attention without positions with a sink
+    and a gate an element; every layer with a routed feed-forward whose active size (top experts and the shared one) is the
+    dense models' ff, between layer norms before and after.  Queries pass a latent of 3/8 of the width.  The key rows are 256
+    numbers (192 + 64 rotated; 256) unless the size says otherwise."""
+    rank = z.get("kv_rank", 192)
+    rotated = {"heads": z["heads"], "dim": z["dim"], "rot_dim": 64, "vdim": z["dim"], "q_rank": z["width"] * 3 // 8, "kv_rank": rank,
+               "scale": (z["dim"] + 64) ** -0.5, "rot": {"base": 500000.0, "dims": 64}}
+    plain = {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "q_rank": z["width"] * 3 // 8,
+             "kv_rank": 256 if rank == 192 else rank, "scale": z["dim"] ** -0.5}
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"] // 6, "limit": 7.0}, "shared": {"ff": z["ff"] // 3, "limit": 7.0},
+           "router": {"experts": 32, "top": 4}}
+    layers = [{"type": "latent_attention", "mixer": dict(plain), "mlp": dict(mlp)} if i % 2 else
+              {"type": "latent_attention_2", "mixer": dict(rotated), "mlp": dict(mlp)} for i in range(z["layers"])]
+    return {"architecture": "Bozavik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 12.0}, "residual_mult": 0.3, "layers": layers}
+
+
+def bozavik_times(args):
+    return design_times(args, "bozavik", (("bozavik", bozavik_config), ("vusalix", vusalix_config), ("qwen3", qwen3_config_like)))
+
+
 def bizepel_times(args):
     return design_times(args, "bizepel", (("bizepel", bizepel_config), ("vusalix", vusalix_config), ("tinuzen", tinuzen_config),
                                           ("qwen3", qwen3_config_like)))
@@ -978,7 +1000,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "timeline", "timeline-prefill", "sample", "attention", "peaks", "sugizen", "tinuzen", "vusalix",
-                             "bizepel"],
+                             "bizepel", "bozavik"],
                     help="a part of the run only (for profiling); the JSON line then holds that part. "
                          "timeline: every kernel of a decode step with its begin and end inside the graph "
                          "(timeline-prefill: of a prompt); "
@@ -988,7 +1010,8 @@ def main():
                          "(two widths, eight layers), with every kernel's time in a prompt and in a decode step; "
                          "tinuzen: the same for the Tinuzen design beside Sugizen and Qwen3; "
                          "vusalix: the same for the Vusalix design beside Sugizen and Qwen3; "
-                         "bizepel: the same for the Bizepel design beside Vusalix, Tinuzen and Qwen3")
+                         "bizepel: the same for the Bizepel design beside Vusalix, Tinuzen and Qwen3; "
+                         "bozavik: the same for the Bozavik design beside Vusalix and Qwen3")
     ap.add_argument("--batch", type=int, default=BATCH, help="sequences of the decode step")
     ap.add_argument("--fast-fill", action="store_true", help="do not run the prompts; mark the cache as filled")
     ap.add_argument("--prompt", type=int, default=PROMPT, help="positions each sequence holds before the timed steps")
@@ -1027,6 +1050,8 @@ def main():
         return vusalix_times(args)
     if args.only == "bizepel":
         return bizepel_times(args)
+    if args.only == "bozavik":
+        return bozavik_times(args)
     if args.config != "8b":
         return run_other(args)
     return run_ours(args)

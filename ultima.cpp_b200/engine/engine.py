@@ -357,7 +357,8 @@ class Engine:
         from ..kernels import attn_tc
         key = [B]
         for g in self.cache.kv_groups:
-            key.append(attn_tc.decode_slices(B, g.need.n_kv_heads, longest, g.need.window))
+            cap = attn_tc.LATENT_SLICE_CAP if g.need.values_in_keys else attn_tc.SLICE_CAP
+            key.append(attn_tc.decode_slices(B, g.need.n_kv_heads, longest, g.need.window, cap=cap))
         return tuple(key)
 
     def _decode_pass(self, slots, new_tokens, before, want_rows, tables, ids_dev=None) -> torch.Tensor:

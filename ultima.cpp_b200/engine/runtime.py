@@ -226,6 +226,10 @@ class Runtime:
         self.launches += 1
         if self.use_tensor_cores and q_lat.dtype == torch.bfloat16:
             from ..kernels import attn_tc
+            if attn_tc.accepts_latent(q_lat, kv, row, rank, n_heads, scale):
+                o = self.arena.alloc((T, n_heads, rank), self.dtype)
+                attn_tc.latent_attention(q_lat, kv, o, batch, n_heads, row, rank, scale, self, window=window, sink_vals=sink_vals)
+                return o
             if attn_tc.accepts(q2, kv, row, n_heads, 1) and attn_tc.LATENT:
                 o = self.arena.alloc((T, n_heads, row), self.dtype)
                 o2 = o.view(T, n_heads * row)

@@ -147,26 +147,96 @@ def accepts(q, kv, head_dim, n_heads, n_kv_heads) -> bool:
 
 
 def decode_slices(n_seqs: int, n_kv_heads: int, longest: int, window, per_sm: int = SLICE_FACTOR,
-                  n_sms: int | None = None) -> int:
+                  n_sms: int | None = None, cap: int = SLICE_CAP) -> int:
     """Slices of the key range, so that a decode step with few sequences still fills the GPU
     (``per_sm`` CTAs an SM; ``n_sms``: the device's multiprocessors, asked of it when not given)."""
     span = longest if not window else min(longest, window + 64)
     tiles = max(1, -(-span // 64))
     ctas = n_seqs * n_kv_heads
     want = -(-per_sm * (n_sms or sm_count()) // ctas)
-    n = max(1, min(want, tiles, SLICE_CAP))
+    n = max(1, min(want, tiles, cap))
     return 1 << (n.bit_length() - 1)            # a power of two: few distinct captured graphs
 
 
-# ULTIMA_ATTN_LATENT=0: latent attention stays on the any-shape kernel
-LATENT = _os.environ.get("ULTIMA_ATTN_LATENT", "1") != "0"
+# ULTIMA_ATTN_LATENT=0: latent attention stays on the any-shape kernel; 1: not on the tcgen05 kernel
+LATENT = int(_os.environ.get("ULTIMA_ATTN_LATENT", "2"))
+LATENT_SLICE_CAP = int(_os.environ.get("ULTIMA_LATENT_SLICE_CAP", "64"))
+LATENT_SOURCE = "attn_latent.cu"
+_latent_libs: dict = {}
 
 
-def latent_needs(row: int, n_heads: int) -> list:
+def latent_fits(row: int, rank: int, n_heads: int) -> bool:
+    """The tcgen05 kernel of latent attention (csrc/attn_latent.cu): rows and values in eights, up to 576 and 512 of them,
+    up to 128 heads."""
+    return LATENT >= 2 and row % 8 == 0 and rank % 8 == 0 and 8 <= rank <= min(row, 512) and row <= 576 and n_heads <= 128
+
+
+def latent_target(row: int):
+    return (LATENT_SOURCE, (f"ROW_BLOCKS={-(-int(row) // 64)}",))
+
+
+def latent_needs(row: int, rank: int, n_heads: int) -> list:
     """The libraries latent attention over key rows of ``row`` numbers uses beyond the any-shape kernel."""
+    if latent_fits(row, rank, n_heads):
+        return [latent_target(row)]
     if LATENT and row % 16 == 0 and 16 <= row <= 256:
         return [target(row)]
     return []
+
+
+def latent_lib(row: int):
+    blocks = -(-int(row) // 64)
+    L = _latent_libs.get(blocks)
+    if L is None:
+        L = build.load(*latent_target(row))
+        L.ub_attn_latent_map_q.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_longlong, c_int]
+        L.ub_attn_latent_map_q.restype = c_int
+        L.ub_attn_latent_map_k.argtypes = [c_void_p, c_void_p, c_longlong, c_int]
+        L.ub_attn_latent_map_k.restype = c_int
+        L.ub_attn_latent.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                     c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p,
+                                     c_void_p, c_void_p]
+        L.ub_attn_latent.restype = c_int
+        if L.ub_attn_latent_row_blocks() != blocks:
+            raise KernelError(f"latent attention library was built for {L.ub_attn_latent_row_blocks()} row blocks, not {blocks}")
+        _latent_libs[blocks] = L
+    return L
+
+
+def accepts_latent(q, kv, row: int, rank: int, n_heads: int, scale: float) -> bool:
+    return (latent_fits(row, rank, n_heads) and scale > 0 and q.dtype == torch.bfloat16 and kv.k.dtype == torch.bfloat16
+            and kv.page == 64 and kv.k.is_contiguous() and q.is_contiguous() and q.data_ptr() % 16 == 0 and kv.k.data_ptr() % 16 == 0)
+
+
+def latent_attention(q, kv, out, batch, n_heads, row, rank, scale, rt, window=None, sink_vals=None, slices: int | None = None):
+    """q [T, heads, row] over one key head whose rows of ``row`` numbers have the values as their leading ``rank`` columns;
+    out [T, heads, rank].  ``sink_vals`` float32 [heads]: one more term exp(sink) in the softmax's sum."""
+    L = latent_lib(row)
+    T = q.shape[0]
+    assert out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape == (T, n_heads, rank)
+    assert sink_vals is None or (sink_vals.dtype == torch.float32 and sink_vals.is_contiguous() and sink_vals.numel() == n_heads)
+    decode = batch.max_new == 1 and batch.n_seqs == T
+    mq = _tc_map(("lq", q.data_ptr(), T, n_heads, row), lambda a: L.ub_attn_latent_map_q(a, q.data_ptr(), T, n_heads, n_heads * row, row))
+    mk = _tc_map(("lk", kv.k.data_ptr(), kv.k.shape[0], row), lambda a: L.ub_attn_latent_map_k(a, kv.k.data_ptr(), kv.k.shape[0], row))
+    part_o = part_ml = None
+    n_slices = 1
+    if decode:
+        parts = -(-rank // 256)
+        n_slices = slices or latent_slices(batch.n_seqs, batch.max_after, window, parts)
+        if n_slices > 1:
+            part_o = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, rank), torch.float32)
+            part_ml = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, 2), torch.float32)
+    rc = L.ub_attn_latent(1 if decode else 0, mq, mk, _ptr(out), n_heads * rank, _ptr(batch.seq_start), _ptr(batch.seq_before),
+                          _ptr(kv.table), kv.table.shape[1], kv.ring, kv.page, batch.n_seqs, batch.max_new, n_heads, row, rank,
+                          int(window or 0), float(scale), _ptr(sink_vals), n_slices, _ptr(part_o), _ptr(part_ml),
+                          _ptr(rt.status[1:2]), _stream())
+    _check(rc, "attn_latent")
+
+
+def latent_slices(n_seqs: int, longest: int, window, parts: int = 1, n_sms: int | None = None) -> int:
+    """Slices of the key range of a latent decode step: a CTA an SM.  What ``decode_slices`` gives with the same cap and more
+    CTAs an SM determines it, so that is what a captured step may be looked up by."""
+    return decode_slices(n_seqs * parts, 1, longest, window, per_sm=1, n_sms=n_sms, cap=LATENT_SLICE_CAP)
 
 
 FUSE_QKV = _os.environ.get("ULTIMA_ATTN_FUSE_QKV", "1") != "0"

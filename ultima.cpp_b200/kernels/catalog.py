@@ -10,11 +10,13 @@ HEAD_DIMS = (16, 32, 48, 64, 80, 96, 112, 128, 256)
 
 
 TC_HEAD_DIMS = (64, 128)          # head sizes the tcgen05 prefill attention is written for
+LATENT_ROW_BLOCKS = (1, 2, 3, 4, 5, 9)       # 64-column blocks of a latent key row (any up to 9 is built on demand)
 
 
 def all_targets() -> list:
     return (list(PLAIN) + [("attn_mma.cu", (f"HEAD_DIM={hd}",)) for hd in HEAD_DIMS]
             + [("attn_tcgen05.cu", (f"HEAD_DIM={hd}",)) for hd in TC_HEAD_DIMS]
+            + [("attn_latent.cu", (f"ROW_BLOCKS={n}",)) for n in LATENT_ROW_BLOCKS]
             + [("decode_stack.cu", (f"HEAD_DIM={hd}",)) for hd in TC_HEAD_DIMS])
 
 

@@ -91,7 +91,7 @@ class LatentAttention(Mixer):
         from ..kernels import attn_tc
         out = [("latent.cu", ()), ("attn_simple.cu", ())]
         if run_dtype == torch.bfloat16:
-            out += attn_tc.latent_needs(self.row, self.nh)
+            out += attn_tc.latent_needs(self.row, self.rank, self.nh)
         return out
 
     def frequencies(self):
