@@ -397,22 +397,21 @@ __global__ void attn_latent_combine_kernel(LatentParams p) {
     const int seq = sh / p.nh, head = sh % p.nh;
     const long long base = (long long)sh * p.n_slices;
     float mm = -INFINITY;
+#pragma unroll 8
     for (int s = 0; s < p.n_slices; ++s) mm = fmaxf(mm, p.part_ml[(base + s) * 2]);
     const float sk = p.sink ? p.sink[head] * LOG2E : -INFINITY;
     mm = fmaxf(mm, sk);
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     float ll = p.sink ? exp2f(sk - mm) : 0.f;
+    if (d >= p.vals) return;
+#pragma unroll 8
     for (int s = 0; s < p.n_slices; ++s) {
         const float ms = p.part_ml[(base + s) * 2];
-        if (ms == -INFINITY) continue;                     // an empty slice
-        const float f = exp2f(ms - mm);
-        ll += f * p.part_ml[(base + s) * 2 + 1];
-        if (d < p.vals) {
-            const float4 o = *reinterpret_cast<const float4*>(p.part_o + (base + s) * p.vals + d);
-            acc.x = fmaf(f, o.x, acc.x); acc.y = fmaf(f, o.y, acc.y); acc.z = fmaf(f, o.z, acc.z); acc.w = fmaf(f, o.w, acc.w);
-        }
+        const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);        // (an empty slice has written zeros)
+        ll = fmaf(f, p.part_ml[(base + s) * 2 + 1], ll);
+        const float4 o = *reinterpret_cast<const float4*>(p.part_o + (base + s) * p.vals + d);
+        acc.x = fmaf(f, o.x, acc.x); acc.y = fmaf(f, o.y, acc.y); acc.z = fmaf(f, o.z, acc.z); acc.w = fmaf(f, o.w, acc.w);
     }
-    if (d >= p.vals) return;
     const float inv = 1.0f / ll;
     const float v[4] = {acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv};
     store_vec<bf16, 4>(p.out + (long long)p.seq_start[seq] * p.o_stride + (long long)head * p.vals + d, v);

@@ -54,12 +54,32 @@ struct GemmParams {
     // 2 the squared rectifier max(v, 0)^2 (whole K only: a slice's partial sum has no activation)
     int unary;
     // every stored result (not the adding epilogue's) times the sigmoid of mul[t * mul_ld + n * mul_col] (null: no gate), n the
-    // result's column: mul_col 1 is a gate an element, 0 one a row
+    // result's column: mul_col 1 is a gate an element, 0 one a row (the interleaved gate product's gates are one a row)
     const float* mul; long long mul_ld; int mul_col;
 };
 
-__device__ __forceinline__ float out_gate(const GemmParams& p, int t, int n) {
-    return p.mul ? 1.0f / (1.0f + __expf(-p.mul[(long long)t * p.mul_ld + (long long)n * p.mul_col])) : 1.0f;
+// The gates of sixteen neighbouring tokens from t on for the result's column n, asked for before anything is stored (a load
+// behind a store would wait for it): one a token (mul_col 0), held by lane c for token c, or one an element, all sixteen here.
+// ``n_ok``: the column exists.
+__device__ __forceinline__ void load_gates(const GemmParams& p, int t, int n, bool n_ok, int lane, float* gv) {
+    if (p.mul_col == 0) {
+        gv[0] = (lane < 16 && t + lane < p.T) ? p.mul[(long long)(t + lane) * p.mul_ld] : 0.f;
+        return;
+    }
+    const float* src = p.mul + (long long)t * p.mul_ld + (long long)n * p.mul_col;
+#pragma unroll
+    for (int c = 0; c < 16; ++c) gv[c] = (n_ok && t + c < p.T) ? src[c * p.mul_ld] : 0.f;
+}
+__device__ __forceinline__ void sigmoid_gates(const GemmParams& p, float* gv) {
+    auto sig = [](float g) { return __fdividef(1.0f, 1.0f + __expf(-g)); };
+    if (p.mul_col == 0) {
+        const float mine = sig(gv[0]);                     // every lane of the warp comes here
+#pragma unroll
+        for (int c = 0; c < 16; ++c) gv[c] = __shfl_sync(0xffffffffu, mine, c);
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 16; ++c) gv[c] = sig(gv[c]);
 }
 
 __device__ __forceinline__ float unary_of(int kind, float v) {
@@ -113,7 +133,10 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
         const uint32_t taddr = tmem_acc + ((uint32_t)(q * 32) << 16) + (uint32_t)c0;
         tmem_ld16(taddr, r);
         if (EPI == EPI_SWIGLU) tmem_ld16(taddr + BN, r2);
+        float gv[16];
+        if (EPI != EPI_ADD && p.mul) load_gates(p, t0 + c0, EPI == EPI_SWIGLU_IL ? 0 : n, n < p.N, lane, gv);
         tmem_ld_wait();
+        if (EPI != EPI_ADD && p.mul) sigmoid_gates(p, gv);
         if (EPI == EPI_SWIGLU_IL) {
             // lanes 64..127 hold "up" of the 64 features whose "gate" lanes 0..63 hold.  The halves
             // swap through shared memory: gate threads finish columns 0..7, up threads 8..15.
@@ -131,7 +154,9 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
                     if (t >= p.T) break;
                     const float own = __uint_as_float(up ? r[8 + c] : r[c]), other = xch[col * 64 + fl];
                     const float g = up ? other : own, u = up ? own : other;
-                    out[(long long)t * p.ldo + f] = from_f32<TO>(gate_product(p, g, u) * out_gate(p, t, f));
+                    float v = gate_product(p, g, u);
+                    if (p.mul) v *= up ? gv[8 + c] : gv[c];
+                    out[(long long)t * p.ldo + f] = from_f32<TO>(v);
                 }
             }
             asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -140,16 +165,20 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
             for (int c = 0; c < 16; ++c) {
                 const int t = t0 + c0 + c;
                 if (t >= p.T) break;
-                const float v = __uint_as_float(r[c]);
+                float v = __uint_as_float(r[c]);
                 TO* dst = out + (long long)t * p.ldo + n;
-                if (EPI == EPI_STORE) *dst = from_f32<TO>(unary_of(p.unary, v) * out_gate(p, t, n));
+                if (EPI == EPI_STORE) {
+                    v = unary_of(p.unary, v);
+                    *dst = from_f32<TO>(p.mul ? v * gv[c] : v);
+                }
                 else if (EPI == EPI_ADD) {
                     // a reduction at the memory side: no load, no wait; one writer an element
                     // unless K is split, so the sum's order is fixed in that case
                     asm volatile("red.global.add.f32 [%0], %1;" ::"l"(dst), "f"(v) : "memory");
                 } else {
                     const float u = __uint_as_float(r2[c]);
-                    *dst = from_f32<TO>(gate_product(p, v, u) * out_gate(p, t, n));
+                    v = gate_product(p, v, u);
+                    *dst = from_f32<TO>(p.mul ? v * gv[c] : v);
                 }
             }
         }
@@ -885,7 +914,7 @@ UB_API int ub_gemm_tc(const void* map_w, const void* map_w2, const void* map_a, 
     if (splits > 1 && (epi == EPI_SWIGLU || epi == EPI_SWIGLU_IL)) return UB_ERR_ARG;
     if (epi == EPI_SWIGLU_IL && (N % 128) != 0) return UB_ERR_ARG;
     if (splits > 1 && epi == EPI_STORE && o_dtype != UB_F32) return UB_ERR_ARG;
-    if (mul && (splits > 1 || epi == EPI_ADD)) return UB_ERR_ARG;
+    if (mul && (splits > 1 || epi == EPI_ADD || (epi == EPI_SWIGLU_IL && mul_col != 0))) return UB_ERR_ARG;
     const int nkb = (K + BK - 1) / BK;
     GemmParams p;
     p.out = out; p.ldo = ldo; p.split_stride = splits > 1 ? split_stride : 0;
@@ -1023,7 +1052,7 @@ UB_API int ub_gemm_tc_pair(const void* map_w, const void* map_a, void* out, int 
     p.kb_per_split = (K + BK - 1) / BK;
     p.atomic = 0; p.share_tail = 0; p.error = error;
     set_gate_constants(p, gate);
-    if (mul && epi == EPI_ADD) return UB_ERR_ARG;
+    if (mul && (epi == EPI_ADD || (epi == EPI_SWIGLU_IL && mul_col != 0))) return UB_ERR_ARG;
     p.mul = mul; p.mul_ld = mul_ld; p.mul_col = mul_col;
     const CUtensorMap* mw = (const CUtensorMap*)map_w;
     const CUtensorMap* ma = (const CUtensorMap*)map_a;

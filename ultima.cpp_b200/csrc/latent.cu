@@ -30,6 +30,7 @@ struct LatentPlace {
     const int* tok_pos; const int* tok_seq;
     int nh, dim, rot, rank;
     float eps;
+    int vec;                                         // the query columns four a thread: sizes and places in fours
 };
 
 template <typename TX, typename TQ, typename TC>
@@ -85,7 +86,28 @@ latent_place_kernel(const TX* __restrict__ x, LatentPlace<TQ, TC> p, PagedKV c) 
         for (int i = tid; i < p.q_rank; i += blockDim.x) p.d_out[t * p.q_rank + i] = from_f32<TQ>(row[i] * inv * p.dw[i]);
     }
     // the query and gate columns, shared out over the token's blocks
-    if (p.q_off >= 0) {
+    if (p.q_off >= 0 && p.vec) {                     // four neighbouring columns a thread: both pairs of a rotated part at once
+        const int qd = p.dim + p.rot, per = qd >> 2;
+        for (int i = blockIdx.y * blockDim.x + tid; i < p.nh * per; i += blockDim.x * gridDim.y) {
+            const int h = i / per, d = (i % per) * 4;
+            float v[4] = {0.f, 0.f, 0.f, 0.f};
+            for (int s = 0; s < p.n_parts; ++s) {
+                float a[4];
+                load_vec<TX, 4>(x + s * p.part_stride + t * p.ldx + p.q_off + h * qd + d, a);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[e] += a[e];
+            }
+            if (d < p.dim) { store_vec<TQ, 4>(p.q_plain + (t * p.nh + h) * p.dim + d, v); continue; }
+            const int e0 = d - p.dim;
+#pragma unroll
+            for (int e = 0; e < 4; e += 2)
+                if (p.cs && e0 + e < p.rd) {
+                    const float u = turned(v[e], v[e + 1], e0 + e), w = turned(v[e + 1], v[e], e0 + e + 1);
+                    v[e] = u; v[e + 1] = w;
+                }
+            store_vec<TQ, 4>(p.q_lat + (t * p.nh + h) * (long long)(p.rank + p.rot) + p.rank + e0, v);
+        }
+    } else if (p.q_off >= 0) {
         const int qd = p.dim + p.rot;
         for (int i = blockIdx.y * blockDim.x + tid; i < p.nh * qd; i += blockDim.x * gridDim.y) {
             const int h = i / qd, d = i % qd;
@@ -120,12 +142,15 @@ UB_API int ub_latent_place(const void* x, int x_dtype, long long ldx, int n_part
     PagedKV c{table, pages_per_seq, ring, page, 1, rank + rot};
     cudaError_t e;
     // for few tokens as many blocks a token as give every thread one query or gate column, up to 16
-    const int cols = (q_off >= 0 ? nh * (dim + rot) : 0) + (g_off >= 0 ? g_width : 0);
+    const size_t xe = x_dtype == UB_F32 ? 4 : 2, qe = act_dtype == UB_F32 ? 4 : 2;
+    const int vec = q_off >= 0 && dim % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && q_off % 4 == 0 && ldx % 4 == 0 && part_stride % 4 == 0 &&
+                    (uintptr_t)x % (4 * xe) == 0 && (uintptr_t)q_plain % (4 * qe) == 0 && (uintptr_t)q_lat % (4 * qe) == 0;
+    const int cols = (q_off >= 0 ? nh * (dim + rot) / (vec ? 4 : 1) : 0) + (g_off >= 0 ? g_width : 0);
     const int sections = (c_off >= 0 && d_off >= 0) ? 2 : 1;
     const int per_token = n_tokens > 64 ? 1 : min(16, max(sections, (cols + 255) / 256));
 #define GO(TX, TQ) do { \
         const LatentPlace<TQ, TQ> p{ldx, part_stride, n_parts, d_off, q_rank, dw, (TQ*)d_out, q_off, (TQ*)q_plain, (TQ*)q_lat, c_off, cw, \
-                                    cs, sn, rd, (TQ*)kcache, g_off, g_width, g_out, tok_pos, tok_seq, nh, dim, rot, rank, eps}; \
+                                    cs, sn, rd, (TQ*)kcache, g_off, g_width, g_out, tok_pos, tok_seq, nh, dim, rot, rank, eps, vec}; \
         e = ub_launch_dependent(latent_place_kernel<TX, TQ, TQ>, dim3(n_tokens, per_token), dim3(256), smem, st, (const TX*)x, p, c); } while (0)
     if (act_dtype != cache_dtype) return UB_ERR_UNSUPPORTED;
     if (x_dtype == UB_F32 && act_dtype == UB_F32) GO(float, float);

@@ -104,6 +104,16 @@ def token_tile(T: int, epilogue: int) -> int:
     return 256 if T > 192 else 128
 
 
+def spread_tile(T: int, N: int, epilogue: int, n_sms: int | None = None) -> int:
+    """The token tile of a product over whole K: ``token_tile``'s, and for a stored result half of it, down to 64, as long as
+    the CTAs then still have an SM each (a router's few output rows against a prompt's many tokens)."""
+    bn = token_tile(T, epilogue)
+    if epilogue == EPI_STORE:
+        while bn > 64 and -(-N // 128) * -(-T // (bn // 2)) <= (n_sms or sm_count()):
+            bn //= 2
+    return bn
+
+
 def cta_slots(bn: int, epilogue: int, n_sms: int | None = None) -> int:
     """CTAs of this kernel that the GPU holds at once: two an SM for token tiles of up to 64 (their
     shared-memory ring is kept to half an SM's), one otherwise.  ``n_sms``: the device's
@@ -162,7 +172,7 @@ def gemm(a, w, out, epilogue, w2, rt, splits: int | None = None, bn: int | None 
     N = w.shape[0]
     assert w.shape[1] == K and out.stride(-1) == 1
     tile_given = bn is not None
-    bn = bn or token_tile(T, epilogue)
+    bn = bn or (token_tile(T, epilogue) if splits else spread_tile(T, N, epilogue))
     s = splits or k_splits(T, N, K, bn, epilogue)
     split_stride = 0
     if out.dim() == 3:
