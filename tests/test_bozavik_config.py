@@ -107,6 +107,14 @@ def test_slices_of_a_latent_decode_step_follow_from_what_a_captured_step_is_look
                 assert seen.setdefault(key, n) == n and 1 <= n <= attn_tc.LATENT_SLICE_CAP
 
 
+def test_a_stored_product_with_few_output_rows_spreads_over_smaller_token_tiles():
+    from ultima_b200.kernels import gemm_tc
+    from ultima_b200.kernels.ops import EPI_ADD, EPI_STORE
+    assert gemm_tc.spread_tile(2048, 33, EPI_STORE, 148) == 64 and gemm_tc.spread_tile(2048, 33, EPI_ADD, 148) == 256
+    assert gemm_tc.spread_tile(2048, 1024, EPI_STORE, 148) == 128 and gemm_tc.spread_tile(2048, 4096, EPI_STORE, 148) == 256
+    assert gemm_tc.spread_tile(20, 33, EPI_STORE, 148) == 32
+
+
 def test_the_bench_models_are_configurations_of_equal_active_size():
     """The models that ``bench.py --only bozavik`` times: chosen and shared experts together have the dense models' inner
     size, and every layer's attention is one the tensor-core kernel takes."""

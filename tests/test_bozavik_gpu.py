@@ -366,6 +366,7 @@ ONE_LAYER = {
     "rotated_whole": _model([_layer(_rotated(4, 16, 24, 40, 32, 0.17, 16, 10000.0))], scale=1.0),
     "rotated_in_part": _model([_layer(_rotated(5, 8, 8, 24, 40, 0.3, 24, 77.0, 10))], width=72),
     "rotated_wide_row": _model([_layer(_rotated(2, 32, 16, 24, 320, 0.1, 32, 500.0))]),
+    "rotated_row_of_sixteens": _model([_layer(_rotated(5, 12, 20, 16, 20, 0.3, 12, 900.0))]),      # the mma.sync kernel's: rank no multiple of 8
     "rotated_no_eights": _model([_layer(_rotated(3, 10, 14, 19, 21, 0.3, 6, 300.0, 4))], width=50),
     "routed": _model([_layer(_SMALL, _moe(10, 3, 24, 1.0, (40, 0.6)))], mult=0.7),
     "routed_no_shared": _model([_layer(_SMALL, _moe(7, 1, 64, 2.0))], width=80),
