@@ -15,6 +15,7 @@ from . import tinuzen  # registers Tinuzen
 from . import vusalix  # registers Vusalix
 from . import bizepel  # registers Bizepel
 from . import bozavik  # registers Bozavik
+from . import demazen  # registers Demazen
 
 for _name in filter(None, (m.strip() for m in os.environ.get("ULTIMA_ARCH_MODULES", "").split(","))):
     importlib.import_module(_name)

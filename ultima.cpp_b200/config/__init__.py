@@ -6,7 +6,8 @@ from .sugizen import SugizenConfig
 from .vusalix import VusalixConfig
 from .bizepel import BizepelConfig
 from .bozavik import BozavikConfig
+from .demazen import DemazenConfig
 
 __all__ = ["ConfigError", "ArchitectureConfig", "ArchitectureEntry", "register_architecture", "find_architecture",
            "known_architectures", "read_config_json", "config_from_dict", "config_from_dir",
-           "Qwen3Config", "SugizenConfig", "VusalixConfig", "BizepelConfig", "BozavikConfig"]
+           "Qwen3Config", "SugizenConfig", "VusalixConfig", "BizepelConfig", "BozavikConfig", "DemazenConfig"]

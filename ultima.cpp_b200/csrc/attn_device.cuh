@@ -11,8 +11,15 @@
 #endif
 static_assert(HEAD_DIM % 16 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= 256, "head size: a multiple of 16 up to 256");
 
-constexpr int HD = HEAD_DIM;
+#ifndef HEAD_DIM_V
+#define HEAD_DIM_V HEAD_DIM
+#endif
+static_assert(HEAD_DIM_V % 16 == 0 && HEAD_DIM_V >= 16 && HEAD_DIM_V <= 256, "value size: a multiple of 16 up to 256");
+
+constexpr int HD = HEAD_DIM;                // queries and keys
+constexpr int HDV = HEAD_DIM_V;             // values
 constexpr int LDS = HD + 8;                 // shared-memory row stride (elements): no bank conflicts for ldmatrix
+constexpr int LDSV = HDV + 8;               // of value rows
 constexpr int KT = 64;                      // keys a tile = positions a page
 constexpr int NTHREADS = 128;
 #ifndef ATTN_DSTAGES
@@ -23,7 +30,7 @@ constexpr int NTHREADS = 128;
 #endif
 constexpr int DSTAGES = ATTN_DSTAGES;       // K/V tiles in the decode kernel's ring
 constexpr int KSTEPS = HD / 16;
-constexpr int DTILES = HD / 8;
+constexpr int DTILES = HDV / 8;
 
 typedef __nv_bfloat16 bf16;
 
@@ -61,10 +68,27 @@ __device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __r
                                              const PagedKV& c, int seq, int kvh, int base, int last_pos, int tid) {
     const long long off = paged_offset(c, seq, base, kvh);            // first position of the page
     constexpr int CH = HD / 8;                                         // 16-byte pieces a row
+    if constexpr (HDV != HD) {                                         // rows of two lengths: the values on their own
+        constexpr int CHV = HDV / 8;
+        const long long off_v = off / HD * HDV;
+        for (int i = tid; i < KT * CH; i += NTHREADS) {
+            const int r = i / CH, ch = i % CH;
+            bf16* kd = Ks + r * LDS + ch * 8;
+            if (base + r <= last_pos) cp_async16(kd, kc + off + (long long)r * HD + ch * 8);
+            else *reinterpret_cast<uint4*>(kd) = make_uint4(0, 0, 0, 0);
+        }
+        for (int i = tid; i < KT * CHV; i += NTHREADS) {
+            const int r = i / CHV, ch = i % CHV;
+            bf16* vd = Vs + r * LDSV + ch * 8;
+            if (base + r <= last_pos) cp_async16(vd, vc + off_v + (long long)r * HDV + ch * 8);
+            else *reinterpret_cast<uint4*>(vd) = make_uint4(0, 0, 0, 0);
+        }
+        return;
+    }
     for (int i = tid; i < KT * CH; i += NTHREADS) {
         const int r = i / CH, ch = i % CH;
         bf16* kd = Ks + r * LDS + ch * 8;
-        bf16* vd = Vs + r * LDS + ch * 8;
+        bf16* vd = Vs + r * LDSV + ch * 8;
         if (base + r <= last_pos) {
             cp_async16(kd, kc + off + (long long)r * HD + ch * 8);
             cp_async16(vd, vc + off + (long long)r * HD + ch * 8);
@@ -109,7 +133,7 @@ __device__ __forceinline__ void weighted_values(float (*o)[4], const float (*s)[
             uint32_t b0, b1, b2, b3;
             const int row = key0 + kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
             const int col = dt * 8 + (lane >> 4) * 8;
-            ldsm_x4_trans(smem_addr(Vs + row * LDS + col), b0, b1, b2, b3);
+            ldsm_x4_trans(smem_addr(Vs + row * LDSV + col), b0, b1, b2, b3);
             mma_bf16(o[dt], a, b0, b1);
             mma_bf16(o[dt + 1], a, b2, b3);
         }
@@ -207,7 +231,7 @@ __device__ __forceinline__ void softmax_step(float (*s)[4], float (*o)[4], float
 }
 
 
-#if HEAD_DIM % 64 == 0
+#if HEAD_DIM % 64 == 0 && HEAD_DIM_V == HEAD_DIM
 #include "tc_common.cuh"
 
 #ifndef ATTN_TSTAGES
@@ -331,4 +355,4 @@ __device__ __forceinline__ void fused_finish(const FusedQKV& f, const float* w, 
     }
 }
 
-#endif   // HEAD_DIM % 64 == 0
+#endif   // HEAD_DIM % 64 == 0 && HEAD_DIM_V == HEAD_DIM

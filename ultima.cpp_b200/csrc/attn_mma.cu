@@ -1,5 +1,6 @@
 // Attention over the paged bfloat16 cache on the tensor cores, for one head size fixed at
-// compile time (-DHEAD_DIM=..., any multiple of 16 up to 256).
+// compile time (-DHEAD_DIM=..., any multiple of 16 up to 256), and one value size where it is another
+// (-DHEAD_DIM_V=..., the same kinds; the prompt and decode kernels on cp.async only).
 //
 // Two kernels share the inner tile code (flash attention: scores, running maximum and sum in
 // float32, probabilities rounded to bfloat16 for the second product):
@@ -29,7 +30,7 @@ struct AttnParams {
     int n_slices;
     // the extended kernels (EXT) only: positions kept visible behind the window, a sink in the softmax's sum,
     // one slope a head (times log2(e)) for the bias by distance, a constant on the output, and one gate an
-    // output element (float32 [tokens, heads * HD], row stride g_stride), whose sigmoid multiplies the output
+    // output element (float32 [tokens, heads * HDV], row stride g_stride), whose sigmoid multiplies the output
     int keep_first, sink;
     const float* slopes;
     float out_scale;
@@ -73,7 +74,7 @@ attn_prefill_kernel(AttnParams p, PagedKV c) {
     pdl_wait();
     bf16* Qs = (bf16*)smem_raw;                    // [64][LDS]
     bf16* Ks = Qs + 64 * LDS;                      // [2][64][LDS]
-    bf16* Vs = Ks + 2 * KT * LDS;                  // [2][64][LDS]
+    bf16* Vs = Ks + 2 * KT * LDS;                  // [2][64][LDSV]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int seq = blockIdx.y, kvh = blockIdx.z;
     const int q0 = p.seq_start[seq], q_len = p.seq_start[seq + 1] - q0, before = p.seq_before[seq];
@@ -121,13 +122,13 @@ attn_prefill_kernel(AttnParams p, PagedKV c) {
     // behind the loop's first barrier)
     const bool bias_here = EXT && p.dist_bias && p.bias_stride > 0;
     if (bias_here) {
-        float* Bs = (float*)(Vs + 2 * KT * LDS);
+        float* Bs = (float*)(Vs + 2 * KT * LDSV);
         for (int i = tid; i < G * p.n_dist; i += NTHREADS) {
             const int d = i / G, g = i % G;
             Bs[g * p.bias_stride + d] = p.dist_bias[(long long)d * p.nh + kvh * G + g];
         }
     }
-    const ScoreTable tb{p.softcap, p.scale, bias_here ? (const float*)(Vs + 2 * KT * LDS) : p.dist_bias, p.n_dist,
+    const ScoreTable tb{p.softcap, p.scale, bias_here ? (const float*)(Vs + 2 * KT * LDSV) : p.dist_bias, p.n_dist,
                         bias_here ? 1 : p.nh, bias_here ? p.bias_stride : 1};
     const ScoreTable* tbp = (EXT && (p.softcap > 0.f || p.dist_bias)) ? &tb : nullptr;
     const int row_head[2] = {bias_here ? row_g[0] : kvh * G + row_g[0], bias_here ? row_g[1] : kvh * G + row_g[1]};
@@ -139,7 +140,7 @@ attn_prefill_kernel(AttnParams p, PagedKV c) {
         const int t = tiles.tile(i);
         const int buf = i & 1;
         if (i + 1 < tiles.n) {
-            load_kv_tile(Ks + (buf ^ 1) * KT * LDS, Vs + (buf ^ 1) * KT * LDS, p.kc, p.vc, c, seq, kvh, tiles.tile(i + 1) * KT, last_pos, tid);
+            load_kv_tile(Ks + (buf ^ 1) * KT * LDS, Vs + (buf ^ 1) * KT * LDSV, p.kc, p.vc, c, seq, kvh, tiles.tile(i + 1) * KT, last_pos, tid);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -147,7 +148,7 @@ attn_prefill_kernel(AttnParams p, PagedKV c) {
         }
         __syncthreads();
         const bf16* K = Ks + buf * KT * LDS;
-        const bf16* V = Vs + buf * KT * LDS;
+        const bf16* V = Vs + buf * KT * LDSV;
         float s[8][4];
         scores<8>(s, Qs, warp * 16, K, 0, lane);
         softmax_step<8, EXT>(s, o, m, l, p.c, row_pos, row_ok, t * KT, p.window, lane, p.keep_first, row_slope, tbp, row_head);
@@ -158,7 +159,7 @@ attn_prefill_kernel(AttnParams p, PagedKV c) {
     for (int r = 0; r < 2; ++r) {
         if (!row_ok[r]) continue;
         const float inv = (EXT ? p.out_scale : 1.0f) / l[r];
-        const long long col = (long long)(kvh * G + row_g[r]) * HD + (lane & 3) * 2;
+        const long long col = (long long)(kvh * G + row_g[r]) * HDV + (lane & 3) * 2;
         bf16* dst = p.out + (long long)(q0 + row_tok[r]) * p.o_stride + col;
         const float* gt = (EXT && p.gate) ? p.gate + (long long)(q0 + row_tok[r]) * p.g_stride + col : nullptr;
 #pragma unroll
@@ -184,7 +185,7 @@ attn_decode_kernel(AttnParams p, PagedKV c) {
     bf16* Qs = (bf16*)smem_raw;                    // [16][LDS]
     bf16* Ks = Qs + 16 * LDS;                      // [DSTAGES][64][LDS]
     bf16* Vs = Ks + DSTAGES * KT * LDS;
-    float* red = ATTN_ALIAS ? (float*)Ks : (float*)(Vs + DSTAGES * KT * LDS);   // [4 warps][16 rows][HD + 2]
+    float* red = ATTN_ALIAS ? (float*)Ks : (float*)(Vs + DSTAGES * KT * LDSV);   // [4 warps][16 rows][HDV + 2]
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int slice = blockIdx.x, seq = blockIdx.y, kvh = blockIdx.z;
     const int G = p.group;
@@ -224,7 +225,7 @@ attn_decode_kernel(AttnParams p, PagedKV c) {
 #pragma unroll
     for (int i = 0; i < DSTAGES - 1; ++i) {
         if (t_lo + i <= t_hi)
-            load_kv_tile(Ks + i * KT * LDS, Vs + i * KT * LDS, p.kc, p.vc, c, seq, kvh, tiles.tile(t_lo + i) * KT, pos, tid);
+            load_kv_tile(Ks + i * KT * LDS, Vs + i * KT * LDSV, p.kc, p.vc, c, seq, kvh, tiles.tile(t_lo + i) * KT, pos, tid);
         cp_async_commit();
     }
     for (int t = t_lo; t <= t_hi; ++t) {
@@ -232,7 +233,7 @@ attn_decode_kernel(AttnParams p, PagedKV c) {
         const int ahead = t + DSTAGES - 1;
         if (ahead <= t_hi) {
             const int nb = (ahead - t_lo) % DSTAGES;
-            load_kv_tile(Ks + nb * KT * LDS, Vs + nb * KT * LDS, p.kc, p.vc, c, seq, kvh, tiles.tile(ahead) * KT, pos, tid);
+            load_kv_tile(Ks + nb * KT * LDS, Vs + nb * KT * LDSV, p.kc, p.vc, c, seq, kvh, tiles.tile(ahead) * KT, pos, tid);
         }
         cp_async_commit();
         cp_async_wait<DSTAGES - 1>();
@@ -240,13 +241,13 @@ attn_decode_kernel(AttnParams p, PagedKV c) {
         float s[2][4];
         scores<2>(s, Qs, 0, Ks + buf * KT * LDS, warp * 16, lane);
         softmax_step<2, EXT>(s, o, m, l, p.c, row_pos, row_ok, tiles.tile(t) * KT + warp * 16, p.window, lane, p.keep_first, row_slope, tbp, row_head);
-        weighted_values<2>(o, s, Vs + buf * KT * LDS, warp * 16, lane);
+        weighted_values<2>(o, s, Vs + buf * KT * LDSV, warp * 16, lane);
         __syncthreads();                             // the slot is filled again at the next step
     }
     cp_async_wait<0>();
     __syncthreads();                                 // K/V no longer needed: the merge buffer lies over them
     // merge the four warps: each has (m, l, o) over its keys
-    constexpr int RS = HD + 2;
+    constexpr int RS = HDV + 2;
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         float* dst = red + ((warp * 16) + (lane >> 2) + r * 8) * RS;
@@ -255,42 +256,42 @@ attn_decode_kernel(AttnParams p, PagedKV c) {
             dst[dt * 8 + (lane & 3) * 2] = o[dt][2 * r];
             dst[dt * 8 + (lane & 3) * 2 + 1] = o[dt][2 * r + 1];
         }
-        if ((lane & 3) == 0) { dst[HD] = m[r]; dst[HD + 1] = l[r]; }
+        if ((lane & 3) == 0) { dst[HDV] = m[r]; dst[HDV + 1] = l[r]; }
     }
     __syncthreads();
-    for (int i = tid; i < G * HD; i += NTHREADS) {
-        const int g = i / HD, d = i % HD;
+    for (int i = tid; i < G * HDV; i += NTHREADS) {
+        const int g = i / HDV, d = i % HDV;
         float mm = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < 4; ++w) mm = fmaxf(mm, red[(w * 16 + g) * RS + HD]);
+        for (int w = 0; w < 4; ++w) mm = fmaxf(mm, red[(w * 16 + g) * RS + HDV]);
         const bool with_sink = EXT && p.sink && p.n_slices == 1;      // (with several slices the sink joins in attn_combine)
         const float sk = with_sink ? sink_log2(p, kvh * G + g) : 0.f;
         if (with_sink) mm = fmaxf(mm, sk);
         float acc = 0.f, ll = with_sink ? exp2f(sk - mm) : 0.f;
 #pragma unroll
         for (int w = 0; w < 4; ++w) {
-            const float mw = red[(w * 16 + g) * RS + HD];
+            const float mw = red[(w * 16 + g) * RS + HDV];
             const float f = mw == -INFINITY ? 0.f : exp2f(mw - mm);
             acc += f * red[(w * 16 + g) * RS + d];
-            ll += f * red[(w * 16 + g) * RS + HD + 1];
+            ll += f * red[(w * 16 + g) * RS + HDV + 1];
         }
         const int head = kvh * G + g;
         if (p.n_slices == 1) {
             float v = acc / ll;
             if constexpr (EXT) {
                 v *= p.out_scale;
-                if (p.gate) v *= 1.0f / (1.0f + __expf(-p.gate[(long long)row * p.g_stride + (long long)head * HD + d]));
+                if (p.gate) v *= 1.0f / (1.0f + __expf(-p.gate[(long long)row * p.g_stride + (long long)head * HDV + d]));
             }
-            p.out[(long long)row * p.o_stride + (long long)head * HD + d] = __float2bfloat16_rn(v);
+            p.out[(long long)row * p.o_stride + (long long)head * HDV + d] = __float2bfloat16_rn(v);
         } else {
             const long long pi = ((long long)seq * p.nh + head) * p.n_slices + slice;
-            p.part_o[pi * HD + d] = acc;
+            p.part_o[pi * HDV + d] = acc;
             if (d == 0) { p.part_ml[pi * 2] = mm; p.part_ml[pi * 2 + 1] = ll; }
         }
     }
 }
 
-// merge the slices of a decode step: grid (sequences * heads), HD threads (rounded up to a warp)
+// merge the slices of a decode step: grid (sequences * heads), HDV threads (rounded up to a warp)
 template <bool EXT>
 __global__ void attn_combine_kernel(AttnParams p) {
     pdl_trigger();
@@ -308,27 +309,28 @@ __global__ void attn_combine_kernel(AttnParams p) {
         const float ms = p.part_ml[(base + s) * 2];
         const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
         ll += f * p.part_ml[(base + s) * 2 + 1];
-        if (d < HD) acc += f * p.part_o[(base + s) * HD + d];
+        if (d < HDV) acc += f * p.part_o[(base + s) * HDV + d];
     }
-    if (d < HD) {
+    if (d < HDV) {
         float v = acc / ll;
         if constexpr (EXT) {
             v *= p.out_scale;
-            if (p.gate) v *= 1.0f / (1.0f + __expf(-p.gate[(long long)p.seq_start[seq] * p.g_stride + (long long)head * HD + d]));
+            if (p.gate) v *= 1.0f / (1.0f + __expf(-p.gate[(long long)p.seq_start[seq] * p.g_stride + (long long)head * HDV + d]));
         }
-        p.out[(long long)p.seq_start[seq] * p.o_stride + (long long)head * HD + d] = __float2bfloat16_rn(v);
+        p.out[(long long)p.seq_start[seq] * p.o_stride + (long long)head * HDV + d] = __float2bfloat16_rn(v);
     }
 }
 
 // ---------------------------------------------------------------------------------------
 UB_API int ub_attn_head_dim() { return HD; }
+UB_API int ub_attn_value_dim() { return HDV; }
 
 // mode 0: prefill kernel (any numbers of new tokens), mode 1: decode kernel (one new token for
-// every sequence, group <= 16).  part_o: float32 [n_seqs, nh, n_slices, HD], part_ml: [.., 2].
+// every sequence, group <= 16).  part_o: float32 [n_seqs, nh, n_slices, HDV], part_ml: [.., 2].
 template <bool EXT>
 static int launch_mma(int mode, AttnParams p, PagedKV c, int n_seqs, int max_new, int nkv, cudaStream_t st) {
     static bool attr_done = false;
-    const size_t sm_pre_plain = (size_t)(64 + 4 * KT) * LDS * sizeof(bf16);
+    const size_t sm_pre_plain = (size_t)((64 + 2 * KT) * LDS + 2 * KT * LDSV) * sizeof(bf16);
     size_t sm_bias = 0;
     p.bias_stride = 0;
     if (EXT && mode == 0 && p.dist_bias) {
@@ -336,7 +338,7 @@ static int launch_mma(int mode, AttnParams p, PagedKV c, int n_seqs, int max_new
         if (need <= (size_t)BIAS_SMEM_MAX) { sm_bias = need; p.bias_stride = bias_stride_for(p.n_dist); }
     }
     const size_t sm_pre = sm_pre_plain + sm_bias;
-    const size_t sm_kv = (size_t)2 * DSTAGES * KT * LDS * sizeof(bf16), sm_red = (size_t)64 * (HD + 2) * sizeof(float);
+    const size_t sm_kv = (size_t)DSTAGES * KT * (LDS + LDSV) * sizeof(bf16), sm_red = (size_t)64 * (HDV + 2) * sizeof(float);
     const size_t sm_dec = (size_t)16 * LDS * sizeof(bf16) + (ATTN_ALIAS ? (sm_kv > sm_red ? sm_kv : sm_red) : sm_kv + sm_red);
     if (!attr_done) {
         cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -358,7 +360,7 @@ static int launch_mma(int mode, AttnParams p, PagedKV c, int n_seqs, int max_new
         cudaError_t e = ub_launch_dependent(attn_decode_kernel<EXT>, grid, dim3(NTHREADS), sm_dec, st, p, c);
         if (e != cudaSuccess) return (int)e;
         if (p.n_slices > 1) {
-            e = ub_launch_dependent(attn_combine_kernel<EXT>, dim3(n_seqs * p.nh), dim3(((HD + 31) / 32) * 32), 0, st, p);
+            e = ub_launch_dependent(attn_combine_kernel<EXT>, dim3(n_seqs * p.nh), dim3(((HDV + 31) / 32) * 32), 0, st, p);
             if (e != cudaSuccess) return (int)e;
         }
     }
@@ -426,7 +428,7 @@ UB_API int ub_attn_mma_ext(int mode, const void* q, long long q_stride, void* ou
 // gives the slot back.  ldmatrix addresses undo the swizzle (16-byte piece c of row r lies at
 // piece c ^ (r % 8)), which also makes them free of bank conflicts.
 // ---------------------------------------------------------------------------------------
-#if HEAD_DIM % 64 == 0
+#if HEAD_DIM % 64 == 0 && HEAD_DIM_V == HEAD_DIM
 
 struct TmaDecodeParams {
     AttnParams a;
@@ -728,7 +730,7 @@ UB_API int ub_attn_decode_tma_qkv(const void* map_k, const void* map_v, const fl
     return decode_tma_launch(map_k, map_v, nullptr, 0, out, o_stride, seq_start, seq_before, table, pages_per_seq,
                              ring, page, n_seqs, nh, nkv, window, scale, n_slices, part_o, part_ml, error, f, st);
 }
-#endif   // HEAD_DIM % 64 == 0
+#endif   // HEAD_DIM % 64 == 0 && HEAD_DIM_V == HEAD_DIM
 
 // ---------------------------------------------------------------------------------------
 // decode attention without any allocation: see attn_noalloc.h
@@ -749,7 +751,7 @@ UB_API int ub_attn_decode_noalloc(const void* q, long long q_stride, void* out, 
     if (n_seqs <= 0) return 0;
     if (n_slices < 1 || nh < 1) return UB_ERR_ARG;
     const long long parts = (long long)n_seqs * nh * n_slices;
-    if (parts * HD > UB_NOALLOC_SCRATCH_O_FLOATS || parts * 2 > UB_NOALLOC_SCRATCH_ML_FLOATS) return UB_ERR_NOALLOC_TOO_LARGE;
+    if (parts * HDV > UB_NOALLOC_SCRATCH_O_FLOATS || parts * 2 > UB_NOALLOC_SCRATCH_ML_FLOATS) return UB_ERR_NOALLOC_TOO_LARGE;
     int dev = -1;
     cudaError_t e = cudaGetDevice(&dev);
     if (e != cudaSuccess) return (int)e;

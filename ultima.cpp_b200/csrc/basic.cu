@@ -12,31 +12,38 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------------------
-// embedding: x[t, :] = float(table[ids[t], :]); a bad id sets *status and writes zeros
+// embedding: x[t, :] = float(table[ids[t], :]) * scale (+ ptab[pos[t], :]); a bad id (or a position outside its table)
+// sets *status and writes zeros
 // ---------------------------------------------------------------------------------------
 template <typename TT>
 __global__ void embed_kernel(const TT* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ x, int width, int vocab, int* status, float scale) {
+                             float* __restrict__ x, int width, int vocab, int* status, float scale,
+                             const TT* __restrict__ ptab, const int* __restrict__ pos, int n_pos) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
-    const int id = ids[t];
-    const bool ok = id >= 0 && id < vocab;
+    const int id = ids[t], at = ptab ? pos[t] : 0;
+    const bool ok = id >= 0 && id < vocab && (!ptab || (at >= 0 && at < n_pos));
     if (!ok && threadIdx.x == 0) atomicExch(status, 1);
     const TT* row = table + (long long)(ok ? id : 0) * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x)
-        x[(long long)t * width + i] = ok ? to_f32<TT>(row[i]) * scale : 0.f;
+    const TT* prow = ptab ? ptab + (long long)(ok ? at : 0) * width : nullptr;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        float v = to_f32<TT>(row[i]) * scale;
+        if (prow) v += to_f32<TT>(prow[i]);
+        x[(long long)t * width + i] = ok ? v : 0.f;
+    }
 }
 
 // The same, eight values a thread and step: rows that begin on 16-byte boundaries.
 template <typename TT>
 __global__ void embed_vec_kernel(const TT* __restrict__ table, const int* __restrict__ ids,
-                                 float* __restrict__ x, int width, int vocab, int* status, float scale) {
+                                 float* __restrict__ x, int width, int vocab, int* status, float scale,
+                                 const TT* __restrict__ ptab, const int* __restrict__ pos, int n_pos) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
-    const int id = ids[t];
-    const bool ok = id >= 0 && id < vocab;
+    const int id = ids[t], at = ptab ? pos[t] : 0;
+    const bool ok = id >= 0 && id < vocab && (!ptab || (at >= 0 && at < n_pos));
     if (!ok && threadIdx.x == 0) atomicExch(status, 1);
     const TT* row = table + (long long)(ok ? id : 0) * width;
     for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
@@ -44,28 +51,35 @@ __global__ void embed_vec_kernel(const TT* __restrict__ table, const int* __rest
         load_vec<TT, 8>(row + i, v);
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[j] = ok ? v[j] * scale : 0.f;
+        if (ptab && ok) {
+            float a[8];
+            load_vec<TT, 8>(ptab + (long long)at * width + i, a);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] += a[j];
+        }
         store_vec<float, 8>(x + (long long)t * width + i, v);
     }
 }
 
 UB_API int ub_embed(const void* table, int table_dtype, const int* ids, float* x, int n_tokens,
-                    int width, int vocab, int* status, float scale, cudaStream_t st) {
+                    int width, int vocab, int* status, float scale, const void* ptab, const int* pos, int n_pos, cudaStream_t st) {
     if (n_tokens <= 0) return 0;
+    if (ptab && !pos) return UB_ERR_ARG;
     cudaError_t e;
-    if (width % 8 == 0 && (((uintptr_t)table | (uintptr_t)x) & 15) == 0 && (table_dtype == UB_F32 || table_dtype == UB_BF16)) {
+    if (width % 8 == 0 && (((uintptr_t)table | (uintptr_t)x | (uintptr_t)ptab) & 15) == 0 && (table_dtype == UB_F32 || table_dtype == UB_BF16)) {
         int vt = 32;
         while (vt < 256 && vt * 16 < width) vt <<= 1;
         if (table_dtype == UB_F32)
-            e = ub_launch_dependent(embed_vec_kernel<float>, dim3(n_tokens), dim3(vt), 0, st, (const float*)table, ids, x, width, vocab, status, scale);
+            e = ub_launch_dependent(embed_vec_kernel<float>, dim3(n_tokens), dim3(vt), 0, st, (const float*)table, ids, x, width, vocab, status, scale, (const float*)ptab, pos, n_pos);
         else
-            e = ub_launch_dependent(embed_vec_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(vt), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale);
+            e = ub_launch_dependent(embed_vec_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(vt), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale, (const __nv_bfloat16*)ptab, pos, n_pos);
         return (int)e;
     }
     const int threads = width >= 1024 ? 256 : 128;
     if (table_dtype == UB_F32)
-        e = ub_launch_dependent(embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, st, (const float*)table, ids, x, width, vocab, status, scale);
+        e = ub_launch_dependent(embed_kernel<float>, dim3(n_tokens), dim3(threads), 0, st, (const float*)table, ids, x, width, vocab, status, scale, (const float*)ptab, pos, n_pos);
     else if (table_dtype == UB_BF16)
-        e = ub_launch_dependent(embed_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale);
+        e = ub_launch_dependent(embed_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, st, (const __nv_bfloat16*)table, ids, x, width, vocab, status, scale, (const __nv_bfloat16*)ptab, pos, n_pos);
     else return UB_ERR_UNSUPPORTED;
     return (int)e;
 }

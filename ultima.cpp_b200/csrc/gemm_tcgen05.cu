@@ -51,7 +51,8 @@ struct GemmParams {
     // is the hard limit max(g', 0) * (u' + shift)
     float act_limit, act_alpha, act_shift;
     // EPI_STORE: what is stored is a function of the sum: 0 the sum itself, 1 the exact GELU 0.5 v (1 + erf(v / sqrt 2)),
-    // 2 the squared rectifier max(v, 0)^2 (whole K only: a slice's partial sum has no activation)
+    // 2 the squared rectifier max(v, 0)^2, 3 the soft cap c tanh(v / c) with c = act_limit (whole K only: a slice's partial
+    // sum has no activation)
     int unary;
     // every stored result (not the adding epilogue's) times the sigmoid of mul[t * mul_ld + n * mul_col] (null: no gate), n the
     // result's column: mul_col 1 is a gate an element, 0 one a row (the interleaved gate product's gates are one a row)
@@ -82,9 +83,10 @@ __device__ __forceinline__ void sigmoid_gates(const GemmParams& p, float* gv) {
     for (int c = 0; c < 16; ++c) gv[c] = sig(gv[c]);
 }
 
-__device__ __forceinline__ float unary_of(int kind, float v) {
+__device__ __forceinline__ float unary_of(int kind, float v, float c) {
     if (kind == 1) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
     if (kind == 2) { const float r = fmaxf(v, 0.f); return r * r; }
+    if (kind == 3) return c * tanhf(v / c);
     return v;
 }
 
@@ -168,7 +170,7 @@ __device__ __forceinline__ void epilogue_tile(const GemmParams& p, uint32_t tmem
                 float v = __uint_as_float(r[c]);
                 TO* dst = out + (long long)t * p.ldo + n;
                 if (EPI == EPI_STORE) {
-                    v = unary_of(p.unary, v);
+                    v = unary_of(p.unary, v, p.act_limit);
                     *dst = from_f32<TO>(p.mul ? v * gv[c] : v);
                 }
                 else if (EPI == EPI_ADD) {

@@ -19,7 +19,8 @@
 // ``mode`` (bits) and ``wscale`` choose another router of the same family: bit 0, s = sigmoid(z) instead of the softmax;
 // bit 1, a group's score is the sum of its two largest choice scores instead of the largest; bit 2, the chosen outputs'
 // weights are divided by their sum (+ 1e-20); bit 3, the scores are the logits themselves and the chosen outputs' weights are the
-// softmax over the chosen logits only; the weights are then multiplied by ``wscale``.
+// softmax over the chosen logits only; the weights are then multiplied by ``wscale``.  Bit 4: the stored vector is a bias of the
+// logits themselves (z + bias is what every score is made of) instead of a correction of the choice.
 // A row of z may have columns behind the router's outputs (another small product of the same input): ``extra`` receives the sum of
 // the K slices of the first of them.
 // Places within a segment are handed out by an atomic counter, so they differ from run to run; every row of a
@@ -36,9 +37,12 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
                                             int keep, float* sc, float* ch, float* gm, int lane, int* idx_t, float* wts_t,
                                             int* counts, int mode, float wscale) {
     float m = -INFINITY;
+    const float* bias = (mode & 16) ? corr : nullptr;
+    if (mode & 16) corr = nullptr;
     for (int i = lane; i < n_out; i += 32) {              // the logits may come as K slices: summed in the slices' order
         float v = zr[i];
         for (int s = 1; s < n_parts; ++s) v += zr[s * part_stride + i];
+        if (bias) v += bias[i];
         sc[i] = v;
         m = fmaxf(m, v);
     }

@@ -3,6 +3,8 @@
 //
 //   layernorm        (x - mean) / sqrt(var + eps) * w (+ b), the variance about the mean; float32 sums
 //   norm_join        x += mult * norm(y) with an RMS or a layer norm of the result's own, y cleared, and in the same pass the
+//   norm_join_two    the same for a sublayer that leaves two results: each through an RMS norm and a factor of its own, their sum
+//                    through one more RMS norm, x += that
 //                    next sublayer's input: nothing, x in the activation type, an RMS norm or a layer norm of the new x
 //   scale_add_norm   x += s * y (s one number a channel), y cleared, and in the same pass the next sublayer's
 //                    input: nothing, x in the activation type, an RMS norm or a layer norm of the new x
@@ -14,7 +16,7 @@
 //                    channel's state has one reader, the thread that convolves it, which then moves it on itself)
 //   take_cols        a column range of a projection row (summed over its K slices), optionally through tanh,
 //                    into the activation type, padded with zeros to an aligned width
-//   unary            the exact (erf) GELU or the square of the rectifier, element by element
+//   unary            the exact (erf) GELU, the square of the rectifier or the soft cap, element by element
 //   side_gate        gelu_tanh(s) * table[token, column range]
 // Sums, norms, the convolution and the activations are float32 whatever the types of input and output.
 #include "common.cuh"
@@ -293,6 +295,128 @@ UB_API int ub_norm_join(float* y, float* x, float mult, const float* aw, const f
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     e = f32 ? ub_launch_dependent(norm_join_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y, x, mult, a, mode, n, (float*)out, width, clear_y)
             : ub_launch_dependent(norm_join_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y, x, mult, a, mode, n, (__nv_bfloat16*)out, width, clear_y);
+    return (int)e;
+}
+
+// ---------------------------------------------------------------------------------------
+// Two results, each normed: z = s1 * y1 / rms(y1) * w1 + s2 * y2 / rms(y2) * w2; x += z, or (with aw) x += z / rms(z) * aw; both
+// results cleared; out (if given) = the new x.
+struct JoinTwo {
+    const float* w1; const float* w2; float s1, s2, eps;
+    const float* aw; float a_eps;
+};
+
+template <typename TO>
+__global__ void norm_join_two_kernel(float* __restrict__ y1, float* __restrict__ y2, float* __restrict__ x, JoinTwo j,
+                                     TO* __restrict__ out, int width) {
+    __shared__ float red[33];
+    pdl_trigger();
+    pdl_wait();
+    float* a = y1 + (long long)blockIdx.x * width;
+    float* b = y2 + (long long)blockIdx.x * width;
+    float* xr = x + (long long)blockIdx.x * width;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) { sa += a[i] * a[i]; sb += b[i] * b[i]; }
+    const float ia = inv_rms(block_sum(sa, red), (float)width, j.eps) * j.s1;
+    const float ib = inv_rms(block_sum(sb, red), (float)width, j.eps) * j.s2;
+    float sz = 0.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {          // (a thread meets its own elements only, here and below)
+        const float z = a[i] * ia * j.w1[i] + b[i] * ib * j.w2[i];
+        a[i] = z;
+        b[i] = 0.f;
+        sz += z * z;
+    }
+    const float iz = j.aw ? inv_rms(block_sum(sz, red), (float)width, j.a_eps) : 1.f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float v = fmaf(a[i] * iz, j.aw ? j.aw[i] : 1.f, xr[i]);
+        xr[i] = v;
+        a[i] = 0.f;
+        if (out) out[(long long)blockIdx.x * width + i] = from_f32<TO>(v);
+    }
+}
+
+// The same with the rows in registers, four neighbouring columns a load (rows of a multiple of 4 columns, up to 256 * 4 * NCH).
+template <typename TO, int NCH>
+__global__ void __launch_bounds__(256)
+norm_join_two_vec_kernel(float* __restrict__ y1, float* __restrict__ y2, float* __restrict__ x, JoinTwo j,
+                         TO* __restrict__ out, int width) {
+    __shared__ float red[33], red2[33];
+    pdl_trigger();
+    const int chunks = width >> 2;
+    float4 w1[NCH], w2[NCH], wa[NCH];
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {                                  // the weights are there before the kernel ahead has ended
+        const int c = threadIdx.x + i * 256;
+        if (c < chunks) {
+            w1[i] = reinterpret_cast<const float4*>(j.w1)[c];
+            w2[i] = reinterpret_cast<const float4*>(j.w2)[c];
+            wa[i] = j.aw ? reinterpret_cast<const float4*>(j.aw)[c] : make_float4(1.f, 1.f, 1.f, 1.f);
+        }
+    }
+    pdl_wait();
+    float4* a = reinterpret_cast<float4*>(y1 + (long long)blockIdx.x * width);
+    float4* b = reinterpret_cast<float4*>(y2 + (long long)blockIdx.x * width);
+    float4* xr = reinterpret_cast<float4*>(x + (long long)blockIdx.x * width);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 u[NCH], v[NCH], r[NCH];
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = threadIdx.x + i * 256;
+        u[i] = c < chunks ? a[c] : zero;
+        v[i] = c < chunks ? b[c] : zero;
+        r[i] = c < chunks ? xr[c] : zero;
+        sa += (u[i].x * u[i].x + u[i].y * u[i].y) + (u[i].z * u[i].z + u[i].w * u[i].w);
+        sb += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    }
+    const float ia = inv_rms(block_sum(sa, red), (float)width, j.eps) * j.s1;
+    const float ib = inv_rms(block_sum(sb, red2), (float)width, j.eps) * j.s2;
+    float sz = 0.f;
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        if (threadIdx.x + i * 256 < chunks) {
+            u[i].x = u[i].x * ia * w1[i].x + v[i].x * ib * w2[i].x;
+            u[i].y = u[i].y * ia * w1[i].y + v[i].y * ib * w2[i].y;
+            u[i].z = u[i].z * ia * w1[i].z + v[i].z * ib * w2[i].z;
+            u[i].w = u[i].w * ia * w1[i].w + v[i].w * ib * w2[i].w;
+            sz += (u[i].x * u[i].x + u[i].y * u[i].y) + (u[i].z * u[i].z + u[i].w * u[i].w);
+        }
+    }
+    const float iz = j.aw ? inv_rms(block_sum(sz, red), (float)width, j.a_eps) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NCH; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < chunks) {
+            const float e[4] = {fmaf(u[i].x * iz, wa[i].x, r[i].x), fmaf(u[i].y * iz, wa[i].y, r[i].y),
+                                fmaf(u[i].z * iz, wa[i].z, r[i].z), fmaf(u[i].w * iz, wa[i].w, r[i].w)};
+            xr[c] = make_float4(e[0], e[1], e[2], e[3]);
+            a[c] = zero;
+            b[c] = zero;
+            if (out) store_vec<TO, 4>(out + (long long)blockIdx.x * width + 4 * c, e);
+        }
+    }
+}
+
+UB_API int ub_norm_join_two(float* y1, float* y2, float* x, const float* w1, const float* w2, float s1, float s2, float eps,
+                            const float* aw, float a_eps, void* out, int out_dtype, int n_rows, int width, cudaStream_t st) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0 || !w1 || !w2) return UB_ERR_ARG;
+    if (out && out_dtype != UB_F32 && out_dtype != UB_BF16) return UB_ERR_UNSUPPORTED;
+    const JoinTwo j{w1, w2, s1, s2, eps, aw, a_eps};
+    const bool f32 = !out || out_dtype == UB_F32;
+    const bool aligned = (((uintptr_t)x | (uintptr_t)y1 | (uintptr_t)y2 | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)aw | (uintptr_t)out) & 15) == 0;
+    cudaError_t e;
+    if (width % 4 == 0 && width <= 256 * 4 * 8 && aligned) {
+        const int nch = (width / 4 + 255) / 256;
+#define GO(NCH) e = f32 ? ub_launch_dependent(norm_join_two_vec_kernel<float, NCH>, dim3(n_rows), dim3(256), 0, st, y1, y2, x, j, (float*)out, width) \
+                        : ub_launch_dependent(norm_join_two_vec_kernel<__nv_bfloat16, NCH>, dim3(n_rows), dim3(256), 0, st, y1, y2, x, j, (__nv_bfloat16*)out, width)
+        if (nch <= 1) GO(1); else if (nch <= 2) GO(2); else if (nch <= 4) GO(4); else GO(8);
+#undef GO
+        return (int)e;
+    }
+    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+    e = f32 ? ub_launch_dependent(norm_join_two_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y1, y2, x, j, (float*)out, width)
+            : ub_launch_dependent(norm_join_two_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y1, y2, x, j, (__nv_bfloat16*)out, width);
     return (int)e;
 }
 
@@ -625,9 +749,9 @@ UB_API int ub_take_cols(const float* x, long long ldx, int n_parts, long long pa
 }
 
 // ---------------------------------------------------------------------------------------
-// kind 1: 0.5 z (1 + erf(z / sqrt 2)); 2: max(z, 0)^2
+// kind 1: 0.5 z (1 + erf(z / sqrt 2)); 2: max(z, 0)^2; 3: c tanh(z / c)
 template <typename TI, typename TO>
-__global__ void unary_kernel(const TI* __restrict__ in, TO* __restrict__ out, long long n, int kind) {
+__global__ void unary_kernel(const TI* __restrict__ in, TO* __restrict__ out, long long n, int kind, float c) {
     pdl_trigger();
     pdl_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -635,16 +759,17 @@ __global__ void unary_kernel(const TI* __restrict__ in, TO* __restrict__ out, lo
     const float z = to_f32<TI>(in[i]);
     float v;
     if (kind == 1) v = 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
-    else { const float p = fmaxf(z, 0.f); v = p * p; }
+    else if (kind == 2) { const float p = fmaxf(z, 0.f); v = p * p; }
+    else v = c * tanhf(z / c);
     out[i] = from_f32<TO>(v);
 }
 
-UB_API int ub_unary(const void* in, int in_dtype, void* out, int out_dtype, long long n, int kind, cudaStream_t st) {
+UB_API int ub_unary(const void* in, int in_dtype, void* out, int out_dtype, long long n, int kind, float c, cudaStream_t st) {
     if (n <= 0) return 0;
-    if (kind != 1 && kind != 2) return UB_ERR_ARG;
+    if (kind < 1 || kind > 3 || (kind == 3 && !(c > 0.f))) return UB_ERR_ARG;
     const dim3 grid((unsigned)((n + 255) / 256)), block(256);
     cudaError_t e;
-#define GO(TI, TO) e = ub_launch_dependent(unary_kernel<TI, TO>, grid, block, 0, st, (const TI*)in, (TO*)out, n, kind)
+#define GO(TI, TO) e = ub_launch_dependent(unary_kernel<TI, TO>, grid, block, 0, st, (const TI*)in, (TO*)out, n, kind, c)
     if (in_dtype == UB_F32 && out_dtype == UB_F32) GO(float, float);
     else if (in_dtype == UB_F32 && out_dtype == UB_BF16) GO(float, __nv_bfloat16);
     else if (in_dtype == UB_BF16 && out_dtype == UB_BF16) GO(__nv_bfloat16, __nv_bfloat16);

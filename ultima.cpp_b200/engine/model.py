@@ -140,6 +140,8 @@ class Model:
         rt.pass_id += 1
         if self._embedding_need is not None:
             x = self.embedding.forward_step(batch, cache.run_cache(len(self.spec.runs), batch.tables), rt)
+        elif getattr(self.embedding, "reads_positions", False):
+            x = self.embedding.forward_step(batch, None, rt)
         else:
             x = self.embedding.forward(batch.tok_ids, rt)
         if TRACE:

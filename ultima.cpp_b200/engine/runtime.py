@@ -124,11 +124,11 @@ class Runtime:
             raise RuntimeError("a wait inside a kernel ran out of time; the step's results are not valid")
 
     # ---- products ----------------------------------------------------------------------
-    def matmul(self, a, w, out, epilogue=ops.EPI_STORE, w2=None, gate=None, unary=0, mul=None):
+    def matmul(self, a, w, out, epilogue=ops.EPI_STORE, w2=None, gate=None, unary=0, mul=None, unary_arg=0.0):
         """out (=, +=) a @ w.T with float32 accumulation; see kernels.ops for the epilogues.  ``gate`` =
         (limit, alpha, shift): the constants of a clamped gate product (tensor-core epilogues only).  ``unary``
-        (ops.UNARY_*): out = f(a @ w.T), the function taken of the float32 sums: in the tensor-core product's storing
-        epilogue, elsewhere by a kernel behind the product.  ``mul`` = (gates, column step): the stored result times a sigmoid
+        (ops.UNARY_*, ``unary_arg`` its constant where it has one): out = f(a @ w.T), the function taken of the float32 sums: in
+        the tensor-core product's storing epilogue, elsewhere by a kernel behind the product.  ``mul`` = (gates, column step): the stored result times a sigmoid
         gate (see ``gemm_tc.mul_args``; tensor-core epilogues only)."""
         self.launches += 1
         if unary and (epilogue != ops.EPI_STORE or gate is not None):
@@ -136,7 +136,7 @@ class Runtime:
         if self.use_tensor_cores and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16:
             from ..kernels import gemm_tc
             if unary:
-                gate = gemm_tc.unary_constants(unary)
+                gate = gemm_tc.unary_constants(unary, unary_arg)
             key = gemm_tc.launch_key(a, w, out, epilogue, w2, self._status_ptr, gate, mul)
             if gemm_tc.relaunch(key):
                 return None
@@ -146,7 +146,7 @@ class Runtime:
             sums = self.arena.alloc(tuple(out.shape), torch.float32)
             ops.gemm_simt(a, w, sums)
             self.launches += 1
-            return ops.unary(sums, out, unary)
+            return ops.unary(sums, out, unary, unary_arg)
         if gate is not None or mul is not None:
             raise ops.KernelError("a clamped gate product, or a gate on the result, is an epilogue of the tensor-core product only")
         if epilogue == ops.EPI_SWIGLU_IL:
@@ -260,11 +260,13 @@ class Runtime:
 
     def attention_fast(self, q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, block=None) -> bool:
         """The tensor-core attention kernels with a block mask (``block`` positions, counted from the
-        sequence's start), where they take the case; False where they do not, and nothing was launched."""
+        sequence's start) or the cache's window, and values of the keys' size or another, where they take the case; False where
+        they do not, and nothing was launched."""
         if not (self.use_tensor_cores and q.dtype == torch.bfloat16):
             return False
         from ..kernels import attn_tc
-        if not attn_tc.accepts(q, kv, head_dim, n_heads, n_kv_heads) or not attn_tc.BLOCK_MASK:
+        if not attn_tc.accepts(q, kv, head_dim, n_heads, n_kv_heads) or not attn_tc.BLOCK_MASK \
+                or not attn_tc.sizes_fit(head_dim, kv.v.shape[-1]):
             return False
         self.launches += 1
         attn_tc.attention(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, self, block=block)

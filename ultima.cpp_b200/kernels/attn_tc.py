@@ -16,15 +16,23 @@ SLICE_CAP = int(_os.environ.get("ULTIMA_SLICE_CAP", "16"))
 _libs: dict = {}
 
 
-def target(head_dim: int):
+def target(head_dim: int, value_dim: int | None = None):
     extra = tuple(x for x in _os.environ.get("ULTIMA_ATTN_DEFINES", "").split(",") if x)
+    if value_dim is not None and value_dim != head_dim:
+        extra = (f"HEAD_DIM_V={int(value_dim)}",) + extra
     return (SOURCE, (f"HEAD_DIM={int(head_dim)}",) + extra)
 
 
-def lib(head_dim: int):
-    L = _libs.get(head_dim)
+def sizes_fit(head_dim: int, value_dim: int) -> bool:
+    """Whether the mma.sync kernels are built for these sizes of queries and keys and of values."""
+    return all(d % 16 == 0 and 16 <= d <= 256 for d in (head_dim, value_dim))
+
+
+def lib(head_dim: int, value_dim: int | None = None):
+    value_dim = value_dim or head_dim
+    L = _libs.get((head_dim, value_dim))
     if L is None:
-        L = build.load(*target(head_dim))
+        L = build.load(*target(head_dim, value_dim))
         L.ub_attn_mma.argtypes = [c_int, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                   c_float, c_int, c_void_p, c_void_p, c_void_p]
@@ -33,9 +41,11 @@ def lib(head_dim: int):
                                                                        c_int, c_void_p, c_void_p]
         L.ub_attn_mma_ext.restype = c_int
         L.ub_attn_head_dim.restype = c_int
-        if L.ub_attn_head_dim() != head_dim:
-            raise KernelError(f"attention library was built for head size {L.ub_attn_head_dim()}, not {head_dim}")
-        if head_dim % 64 == 0:
+        L.ub_attn_value_dim.restype = c_int
+        if L.ub_attn_head_dim() != head_dim or L.ub_attn_value_dim() != value_dim:
+            raise KernelError(f"attention library was built for head size {L.ub_attn_head_dim()} (values {L.ub_attn_value_dim()}), not "
+                              f"{head_dim} ({value_dim})")
+        if head_dim % 64 == 0 and value_dim == head_dim:
             L.ub_attn_map_kv.argtypes = [c_void_p, c_void_p, c_longlong, c_int]
             L.ub_attn_map_kv.restype = c_int
             L.ub_attn_decode_tma.argtypes = [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p,
@@ -47,7 +57,7 @@ def lib(head_dim: int):
                                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                                  c_int, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
             L.ub_attn_decode_tma_qkv.restype = c_int
-        _libs[head_dim] = L
+        _libs[(head_dim, value_dim)] = L
     return L
 
 
@@ -302,14 +312,17 @@ def _mask_arg(kv, block) -> int:
 def attention(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, slices: int | None = None,
               kernel: str | None = None, block: int | None = None):
     """kernel: None picks (tcgen05 for prompts where it fits, mma.sync otherwise); "mma" forces the latter.
-    ``block``: mask by blocks of this many positions instead of by the cache's window."""
-    L = lib(head_dim)
+    ``block``: mask by blocks of this many positions instead of by the cache's window.  Values may have another size than
+    keys (the mma.sync kernels then)."""
+    value_dim = kv.v.shape[-1]
+    same = value_dim == head_dim
+    L = lib(head_dim, value_dim)
     mask = _mask_arg(kv, block)
     reach = block or kv.window                       # how far back a token looks at most (None: to the start)
     assert out.dtype == torch.bfloat16 and out.stride(1) == 1
     group = n_heads // n_kv_heads
     decode = batch.max_new == 1 and group <= 16
-    tc_ok = (kernel != "mma" and tcgen05_fits(head_dim, n_heads, n_kv_heads) and out.stride(0) % 8 == 0
+    tc_ok = (same and kernel != "mma" and tcgen05_fits(head_dim, n_heads, n_kv_heads) and out.stride(0) % 8 == 0
              and out.data_ptr() % 16 == 0 and kv.k.is_contiguous() and kv.v.is_contiguous())
     if tc_ok and not decode:
         return run_tcgen05(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, False, mask=mask)
@@ -318,12 +331,12 @@ def attention(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, slice
         return run_tcgen05(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, True, n, mask=mask)
     part_o = part_ml = None
     n_slices = 1
-    tma = (decode and head_dim % 64 == 0 and kernel in (None, "tma") and (USE_TMA_DECODE or kernel == "tma")
+    tma = (same and decode and head_dim % 64 == 0 and kernel in (None, "tma") and (USE_TMA_DECODE or kernel == "tma")
            and kv.k.is_contiguous() and kv.v.is_contiguous())
     if decode:
         n_slices = slices or decode_slices(batch.n_seqs, n_kv_heads, batch.max_after, reach)
         if n_slices > 1:
-            part_o = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, head_dim), torch.float32)
+            part_o = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, value_dim), torch.float32)
             part_ml = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, 2), torch.float32)
     if tma:
         mk = _tc_map(("kvd", kv.k.data_ptr(), kv.k.shape[0], n_kv_heads, head_dim),

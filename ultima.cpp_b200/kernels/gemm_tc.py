@@ -281,10 +281,10 @@ def accepts_grouped(a, w, out, epilogue, w2=None) -> bool:
     return epilogue == EPI_STORE and out.dtype in (torch.bfloat16, torch.float32)
 
 
-def unary_constants(kind: int):
-    """The constants that make a storing product store a function of its sums: 1 the exact GELU, 2 the squared rectifier
-    (whole K only); they travel where a gate product's constants do."""
-    return (float("inf"), 1.0, 0.0, float(kind))
+def unary_constants(kind: int, arg: float = 0.0):
+    """The constants that make a storing product store a function of its sums: 1 the exact GELU, 2 the squared rectifier,
+    3 the soft cap arg * tanh(z / arg) (whole K only); they travel where a gate product's constants do."""
+    return (float(arg) if kind == 3 else float("inf"), 1.0, 0.0, float(kind))
 
 
 def grouped(a, w, out, plan, epilogue, w2, rt, unary: int = 0, gate=None):

@@ -97,7 +97,7 @@ def _declare(lib, source: str) -> None:
     P, I, L, F, U = c_void_p, c_int, c_longlong, c_float, c_ulonglong
     sigs = {
         "basic.cu": {
-            "ub_embed": [P, I, P, P, I, I, I, P, F, P],
+            "ub_embed": [P, I, P, P, I, I, I, P, F, P, P, I, P],
             "ub_rmsnorm": [P, P, P, P, I, I, I, F, P],
             "ub_qk_prepare": [P, I, I, L, P, I, L, P, P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, I, I, P, P, L, P],
             "ub_rotate_pairs": [P, I, L, I, I, I, P, P, P, I, I, P],
@@ -144,12 +144,19 @@ def _declare(lib, source: str) -> None:
                    "ub_mamba1_scan_staged": [P, I, P, P, P, L, I, I, P, P, P, L, I, L, P, I, P, P, P, I, I, I, I, P, P]},
         "rowwise.cu": {"ub_layernorm": [P, P, P, P, I, P, I, I, F, P],
                        "ub_norm_join": [P, P, F, P, P, F, I, I, P, P, F, P, I, I, I, I, P],
+                       "ub_norm_join_two": [P, P, P, P, P, F, F, F, P, F, P, I, I, I, P],
                        "ub_scale_add_norm": [P, P, P, I, P, P, F, P, I, I, I, I, P],
                        "ub_causal_conv": [P, I, L, I, L, I, P, P, P, I, P, P, P, P, I, L, I, I, I, I, I, I, I, I, P, P, P, P],
                        "ub_causal_conv_state": [P, I, L, I, L, I, P, P, P, P, I, I, I, P],
                        "ub_take_cols": [P, L, I, L, I, I, I, P, I, L, I, I, P],
-                       "ub_unary": [P, I, P, I, L, I, P],
+                       "ub_unary": [P, I, P, I, L, I, F, P],
                        "ub_side_gate": [P, L, P, I, L, I, P, I, P, I, L, I, I, I, P]},
+        "linear.cu": {"ub_lin_decay": [P, L, I, L, P, P, P, P, I, F, P],
+                      "ub_lin_gates": [P, L, I, L, P, P, P, F, P, P, P, I, P, P, P, P],
+                      "ub_lin_scan": [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, P],
+                      "ub_lin_scan_cols": [I],
+                      "ub_lin_finish": [P, P, L, P, P, P, I, I, P, I, I, F, F, F, P],
+                      "ub_lin_step": [P, L, I, L, P, P, P, F, P, P, F, P, P, P, P, P, P, I, I, P, I, I, F, F, F, P]},
         "sampling.cu": {"ub_sample": [P, L, P, I, I, P, P, P, P, P, U, P, P, I, P], "ub_sample_params_size": []},
     }.get(source, {})
     for name, args in sigs.items():
@@ -159,14 +166,19 @@ def _declare(lib, source: str) -> None:
 
 
 # ---------------------------------------------------------------------------------------
-def embed(table, ids, out, status, scale=1.0):
-    """out[t, :] = scale * table[ids[t], :] as float32; a bad id raises ``status`` (int32[1])."""
-    _need_cuda(table, ids, out, status)
+def embed(table, ids, out, status, scale=1.0, pos_table=None, positions=None):
+    """out[t, :] = scale * table[ids[t], :] (+ pos_table[positions[t], :]) as float32; a bad id, or a position outside the
+    table, raises ``status`` (int32[1])."""
+    _need_cuda(table, ids, out, status, pos_table, positions)
     T, width = out.shape
     assert out.dtype == torch.float32 and ids.dtype == torch.int32 and out.is_contiguous()
     assert table.is_contiguous() and table.shape[1] == width
+    if pos_table is not None:
+        assert pos_table.is_contiguous() and pos_table.shape[1] == width and pos_table.dtype == table.dtype
+        assert positions.dtype == torch.int32 and positions.numel() == T
     _check(_lib("basic.cu").ub_embed(_ptr(table), _code(table), _ptr(ids), _ptr(out), T, width,
-                                     table.shape[0], _ptr(status), float(scale), _stream()), "embed")
+                                     table.shape[0], _ptr(status), float(scale), _ptr(pos_table), _ptr(positions),
+                                     0 if pos_table is None else pos_table.shape[0], _stream()), "embed")
 
 
 def embed_pairs(table, pairs, ids, batch, last, out, status, scale, buckets, mul_prev, mul_cur):
@@ -566,7 +578,7 @@ def gemm_grouped(a, w, out, tiles, n_tiles, src_rows, max_tiles, epilogue=EPI_ST
 ROUTE_TILE = 64          # sorted rows a tile of the grouped products
 
 
-ROUTE_SIGMOID, ROUTE_GROUP_TOP2, ROUTE_NORMALISE, ROUTE_LOGITS = 1, 2, 4, 8      # bits of a router's ``mode`` (csrc/routed.cu)
+ROUTE_SIGMOID, ROUTE_GROUP_TOP2, ROUTE_NORMALISE, ROUTE_LOGITS, ROUTE_LOGIT_BIAS = 1, 2, 4, 8, 16      # bits of a router's ``mode`` (csrc/routed.cu)
 
 
 def _router_columns(z, extra):
@@ -832,6 +844,132 @@ def delta_finish(o, gate_pre, weight, out, H, E, eps, silu_gate=False):
 
 
 # ---------------------------------------------------------------------------------------
+# recurrent layers whose state decays and takes up k v^T (csrc/linear.cu)
+class LinForm:
+    """The sizes of such a layer and the columns of its projection row: ``offs`` = (q, k, v, output gate, first gate columns,
+    second gate columns).  Head form: the input gate's and the forget gate's H columns; channel form: the ``rank`` low-rank
+    columns of the decay."""
+
+    def __init__(self, H, D, E, offs, rank=0, head_form=False):
+        self.H, self.D, self.E, self.rank, self.head_form = int(H), int(D), int(E), int(rank), bool(head_form)
+        q, k, v, g, a, b = (int(o) for o in offs)
+        self.ints = (c_int * 11)(self.H, self.D, self.E, q, k, v, g, a, b, self.rank, 1 if head_form else 0)
+        self.cols = max(q + H * D, k + H * D, v + H * E, g + H * E, a + (H if head_form else rank), b + (H if head_form else 0))
+
+
+def _lin_in(p, form):
+    assert p.dtype == torch.float32 and p.stride(-1) == 1 and p.shape[-1] >= form.cols
+    return _parts_of(p)
+
+
+def lin_decay(p, form, up, bias, dec, tau):
+    """dec [T, H * D] = sigmoid(low @ up + bias)^(1 / tau), low the low-rank columns of the projection rows p (float32 [T, N] or
+    [parts, T, N], summed), up float32 [rank, H * D]."""
+    _need_cuda(p, up, bias, dec)
+    T, ldp, n_parts, part_stride = _lin_in(p, form)
+    C = form.H * form.D
+    for t, shape in ((up, (form.rank, C)), (bias, (C,)), (dec, (T, C))):
+        assert t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == shape
+    _check(_lib("linear.cu").ub_lin_decay(_ptr(p), ldp, n_parts, part_stride, form.ints, _ptr(up), _ptr(bias), _ptr(dec), T,
+                                          float(tau), _stream()), "lin_decay")
+
+
+def lin_gates(p, form, b_in, b_forget, cap, m, batch, keep, put, floor):
+    """The exponential gates of every token (float32 [T, H] each: keep, put, floor) from the running maximum ``m`` float32
+    [slots, H], which moves on; see csrc/linear.cu."""
+    _need_cuda(p, b_in, b_forget, m, keep, put, floor)
+    T, ldp, n_parts, part_stride = _lin_in(p, form)
+    for t in (b_in, b_forget, m, keep, put, floor):
+        assert t.dtype == torch.float32 and t.is_contiguous()
+    assert b_in.numel() == b_forget.numel() == form.H and m.shape[1] == form.H
+    assert keep.shape == put.shape == floor.shape == (T, form.H)
+    _check(_lib("linear.cu").ub_lin_gates(_ptr(p), ldp, n_parts, part_stride, form.ints, _ptr(b_in), _ptr(b_forget), float(cap),
+                                          _ptr(m), _ptr(batch.seq_start), _ptr(batch.seq_slot), batch.n_seqs, _ptr(keep), _ptr(put),
+                                          _ptr(floor), _stream()), "lin_gates")
+
+
+LIN_CHUNK = 64              # the fewest tokens a chunk of the scan has
+LIN_BLOCKS = 6              # blocks an SM the scan is cut into chunks for
+
+
+def lin_chunks(form, n_seqs: int, max_new: int, n_sms: int | None = None):
+    """(chunks, tokens a chunk) of a step whose longest sequence brings ``max_new`` tokens: as many chunks as fill the GPU, and
+    none at all where cutting would not pay for doing the state's update twice."""
+    cols = 64 if form.D <= 128 else 32
+    blocks = n_seqs * form.H * -(-form.E // cols)
+    want = -(-LIN_BLOCKS * (n_sms or sm_count()) // blocks)
+    n = min(want, max_new // LIN_CHUNK, 65535 // max(1, n_seqs))
+    if n < 4:
+        return 1, max(1, max_new)
+    chunk = -(-max_new // n)
+    chunk = -(-chunk // 8) * 8
+    return -(-max_new // chunk), chunk
+
+
+def lin_scan(p, form, dec, put, out, S, n, batch, work=None, decay=None, chunks=(1, 1)):
+    """The recurrence over a step's tokens from the slots' state S float32 [slots, H, D, E] (head form: n float32 [slots, H, D]
+    too), which moves on.  p float32 [T, N]; dec: decays float32 [T, H * D], or the head form's keep [T, H] with ``put``
+    [T, H].  out float32 [T, H, E] (head form [T, H, E + 1], n.q in the last column).  ``chunks`` = (number, tokens each) with
+    ``work`` float32 [number, seqs, H, D, E or E + 1] and ``decay`` float32 [number, seqs, H, D] ([number, seqs, H])."""
+    _need_cuda(p, dec, put, out, S, n, work, decay)
+    T, ldp, n_parts, _ = _lin_in(p, form)
+    H, D, E = form.H, form.D, form.E
+    EW = E + 1 if form.head_form else E
+    assert n_parts == 1 and p.dim() == 2
+    for t in (dec, put, out, S, n, work, decay):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    assert tuple(S.shape[1:]) == (H, D, E) and out.numel() == T * H * EW and dec.numel() == T * H * (1 if form.head_form else D)
+    if form.head_form:
+        assert put.shape == dec.shape and tuple(n.shape[1:]) == (H, D)
+    count, size = chunks
+    if count > 1:
+        assert work.numel() >= count * batch.n_seqs * H * D * EW and count * size >= batch.max_new
+        assert decay.numel() >= count * batch.n_seqs * H * (1 if form.head_form else D)
+    _check(_lib("linear.cu").ub_lin_scan(_ptr(p), ldp, form.ints, _ptr(dec), _ptr(put), _ptr(out), _ptr(S), _ptr(n), _ptr(work),
+                                         _ptr(decay), _ptr(batch.seq_start), _ptr(batch.seq_slot), batch.n_seqs, int(count), int(size),
+                                         _stream()), "lin_scan")
+
+
+def lin_finish(o, p, form, floor, weight, out, q_scale, eps, out_scale=1.0, silu_gate=False):
+    """out [T, H * E] = norm over each head of q_scale * o (head form: of what is left of it behind the division by
+    max(|q_scale n.q|, floor) + 1e-6), times ``weight`` ([E] shared by the heads or [H * E]), the sigmoid (``silu_gate``: SiLU) of the
+    output gate's columns of p, and out_scale."""
+    _need_cuda(o, p, floor, weight, out)
+    T, ldp, n_parts, _ = _lin_in(p, form)
+    H, E = form.H, form.E
+    assert n_parts == 1 and o.dtype == torch.float32 and o.is_contiguous() and o.numel() == T * H * (E + 1 if form.head_form else E)
+    assert floor is None or (floor.dtype == torch.float32 and floor.is_contiguous() and floor.numel() == T * H)
+    assert weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() in (E, H * E)
+    assert out.is_contiguous() and tuple(out.shape) == (T, H * E)
+    _check(_lib("linear.cu").ub_lin_finish(_ptr(o), _ptr(p), ldp, form.ints, _ptr(floor), _ptr(weight),
+                                           1 if weight.numel() == H * E and H > 1 else 0, 1 if silu_gate else 0, _ptr(out), _code(out),
+                                           T, float(q_scale), float(eps), float(out_scale), _stream()), "lin_finish")
+
+
+def lin_step(p, form, state, batch, weight, out, q_scale, eps, out_scale=1.0, silu_gate=False, decay=None, gates=None):
+    """A step of one token a sequence in one kernel, from the projection rows p (float32 [T, N] or [parts, T, N], summed) to
+    out [T, H * E].  ``state``: (S,) with ``decay`` = (up, bias, tau), or (S, n, m) with ``gates`` = (input bias, forget bias, cap)."""
+    T, ldp, n_parts, part_stride = _lin_in(p, form)
+    H, D, E = form.H, form.D, form.E
+    S, n, m = (tuple(state) + (None, None))[:3]
+    up, bias, tau = decay if decay is not None else (None, None, 0.0)
+    bi, bf, cap = gates if gates is not None else (None, None, 0.0)
+    _need_cuda(p, S, n, m, up, bias, bi, bf, weight, out)
+    for t in (S, n, m, up, bias, bi, bf, weight):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    assert batch.n_seqs == T and batch.max_new == 1 and tuple(S.shape[1:]) == (H, D, E)
+    assert (gates is not None) == form.head_form and (decay is not None) != form.head_form
+    if form.head_form:
+        assert tuple(n.shape[1:]) == (H, D) and tuple(m.shape[1:]) == (H,) and bi.numel() == bf.numel() == H
+    else:
+        assert tuple(up.shape) == (form.rank, H * D) and bias.numel() == H * D
+    assert weight.numel() in (E, H * E) and out.is_contiguous() and tuple(out.shape) == (T, H * E)
+    _check(_lib("linear.cu").ub_lin_step(_ptr(p), ldp, n_parts, part_stride, form.ints, _ptr(up), _ptr(bias), float(tau), _ptr(bi),
+                                         _ptr(bf), float(cap), _ptr(S), _ptr(n), _ptr(m), _ptr(batch.seq_start), _ptr(batch.seq_slot),
+                                         _ptr(weight), 1 if weight.numel() == H * E and H > 1 else 0, 1 if silu_gate else 0, _ptr(out),
+                                         _code(out), T, float(q_scale), float(eps), float(out_scale), _stream()), "lin_step")
+
+
 # ---------------------------------------------------------------------------------------
 # row-wise kernels of a stream with scaled sublayers and input convolutions (csrc/rowwise.cu)
 def layernorm(x, weight, out, eps, rows=None, bias=None):
@@ -865,6 +1003,22 @@ def norm_join(y, x, mult, after, mode=NEXT_NONE, then=None, out=None, clear_y=Tr
     _check(_lib("rowwise.cu").ub_norm_join(_ptr(y), _ptr(x), float(mult), _ptr(aw), _ptr(ab), float(a_eps), 1 if kind == NEXT_LAYER else 0,
                                            int(mode), _ptr(nw), _ptr(nb), float(n_eps), _ptr(out),
                                            _code(out) if out is not None else F32, T, width, 1 if clear_y else 0, _stream()), "norm_join")
+
+
+def norm_join_two(y1, y2, x, weights, scales, eps, after=None, out=None):
+    """x += f(scales[0] * rms_norm(y1, weights[0]) + scales[1] * rms_norm(y2, weights[1])), y1 and y2 cleared; f: one more RMS norm,
+    ``after`` = (weight, eps), or nothing.  ``out`` receives the new x in its own type."""
+    aw, a_eps = after if after is not None else (None, 0.0)
+    _need_cuda(y1, y2, x, weights[0], weights[1], aw, out)
+    T, width = x.shape
+    for v in (y1, y2, x):
+        assert v.dtype == torch.float32 and v.is_contiguous() and v.shape == x.shape
+    for v in (weights[0], weights[1], aw):
+        assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == width)
+    assert out is None or (out.is_contiguous() and tuple(out.shape) == (T, width))
+    _check(_lib("rowwise.cu").ub_norm_join_two(_ptr(y1), _ptr(y2), _ptr(x), _ptr(weights[0]), _ptr(weights[1]), float(scales[0]),
+                                               float(scales[1]), float(eps), _ptr(aw), float(a_eps), _ptr(out),
+                                               _code(out) if out is not None else F32, T, width, _stream()), "norm_join_two")
 
 
 def scale_add_norm(y, scale, x, mode=NEXT_NONE, norm_weight=None, eps=0.0, out=None, clear_y=True, norm_bias=None):
@@ -945,13 +1099,14 @@ def take_cols(x, col_off, n, out, tanh=False):
                                            _code(out), out.stride(0), out.shape[1], T, _stream()), "take_cols")
 
 
-UNARY_GELU_ERF, UNARY_RELU_SQUARED = 1, 2
+UNARY_GELU_ERF, UNARY_RELU_SQUARED, UNARY_SOFTCAP = 1, 2, 3
 
 
-def unary(x, out, kind):
+def unary(x, out, kind, arg=0.0):
+    """out = f(x) element by element, f one of UNARY_*; ``arg``: the cap of UNARY_SOFTCAP, arg * tanh(x / arg)."""
     _need_cuda(x, out)
     assert x.is_contiguous() and out.is_contiguous() and x.shape == out.shape
-    _check(_lib("rowwise.cu").ub_unary(_ptr(x), _code(x), _ptr(out), _code(out), x.numel(), int(kind), _stream()), "unary")
+    _check(_lib("rowwise.cu").ub_unary(_ptr(x), _code(x), _ptr(out), _code(out), x.numel(), int(kind), float(arg), _stream()), "unary")
 
 
 def side_gate(s, table, col0, ids, out, dim):

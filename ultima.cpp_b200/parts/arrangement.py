@@ -41,7 +41,8 @@ class _NormAfter(Arrangement):
     here that is a cleared float32 buffer y, which the norm then folds into x.  The same kernel writes
     the next sublayer's input (x in the activation type) and clears y again, and both buffers are kept
     from layer to layer of a pass, so a layer costs no conversion or clearing kernel of its own after
-    the first."""
+    the first.  A mixer that leaves two results (``apart``) gets a second such buffer, and its own joining kernel
+    applies this norm behind its own."""
 
     def _buffers(self, x, rt):
         carry = getattr(rt, "_norm_after_carry", None)
@@ -55,15 +56,29 @@ class _NormAfter(Arrangement):
             h = rt.arena.alloc(tuple(x.shape), rt.dtype)
             rt.launches += 1
             ops.convert(x, h)
-        rt._norm_after_carry = ((rt.pass_id, x.data_ptr(), tuple(x.shape)), h, y)
+        rt._norm_after_carry = [(rt.pass_id, x.data_ptr(), tuple(x.shape)), h, y, None]
         return h, y
+
+    def _second(self, x, rt):
+        """One more cleared buffer of x's shape, made at the first layer of a pass that asks for it."""
+        carry = rt._norm_after_carry
+        if carry[3] is None:
+            carry[3] = rt.arena.alloc(tuple(x.shape), x.dtype)
+            carry[3].zero_()
+        return carry[3]
 
     def run(self, layer, x, batch, cache, rt):
         h, y = self._buffers(x, rt)
         hn = None if h is x else h
-        mark = rt.arena.mark()
-        layer.mixer.forward(h, y, batch, cache, rt)
-        layer.mixer_norm.add_normed(y, x, rt, h=hn, clear=True)
+        if getattr(layer.mixer, "apart", False) and layer.mixer_norm.kind == "rms":
+            y2 = self._second(x, rt)
+            mark = rt.arena.mark()
+            layer.mixer.forward_apart(h, y, y2, batch, cache, rt)
+            layer.mixer.join(y, y2, x, rt, after=(layer.mixer_norm.weight, layer.mixer_norm.eps), h=hn)
+        else:
+            mark = rt.arena.mark()
+            layer.mixer.forward(h, y, batch, cache, rt)
+            layer.mixer_norm.add_normed(y, x, rt, h=hn, clear=True)
         rt.arena.reset(mark)
         ff = getattr(layer, "feed_forward", None)
         if ff is not None:

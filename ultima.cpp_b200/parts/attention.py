@@ -115,6 +115,9 @@ class Attention(Mixer):
         self.extended = (self.norm_whole or self.keep_first > 0 or self.distance_slope is not None or self.sink
                          or self.values_are_keys or self.wide_gate or self.out_scale != 1.0 or self.softcap is not None
                          or self.distance_buckets is not None)
+        # of these, what the attention itself has to know (the others are the placement's)
+        self.score_options = (self.keep_first > 0 or self.distance_slope is not None or self.sink or self.wide_gate
+                              or self.out_scale != 1.0 or self.softcap is not None or self.distance_buckets is not None)
         self._table_options = self.softcap is not None or self.distance_buckets is not None or self.learned_sink
         self.in_bias, self.conv = bool(in_bias), int(conv or 0)
         self.value_mix, self.value_mix_key = value_mix, str(value_mix_key)
@@ -177,15 +180,15 @@ class Attention(Mixer):
             return [("attn_simple.cu", ())] + shaping
         if self.general:
             out = [("attn_simple.cu", ())] + shaping
-            if self.extended:
+            if self.score_options:
                 if self._fast_extended() and attn_tc.EXTENDED:
                     out.append(attn_tc.target(self.hd))
                     if self.hd in catalog.TC_HEAD_DIMS and not self.window and self.distance_slope is None:
                         out.append(attn_tc.tc_target(self.hd))
                 return out
             if self._fast_attention() and attn_tc.BLOCK_MASK:
-                out.append(attn_tc.target(self.hd))
-                if self.hd in catalog.TC_HEAD_DIMS:
+                out.append(attn_tc.target(self.hd, self.hdv))
+                if self.hd in catalog.TC_HEAD_DIMS and self.hdv == self.hd:
                     out.append(attn_tc.tc_target(self.hd))
             return out
         if self.hd % 16 == 0 and 16 <= self.hd <= 256:
@@ -196,14 +199,15 @@ class Attention(Mixer):
         return [("attn_simple.cu", ())]
 
     def _fast_attention(self) -> bool:
-        """Whether a general layer's attention itself can still go to the tensor-core kernels: equal head
-        sizes of a kind they take; the block mask they know, the gate is applied behind them."""
-        return self.hdv == self.hd and self.hd % 16 == 0 and 16 <= self.hd <= 256 and not self.extended
+        """Whether a general layer's attention itself can still go to the tensor-core kernels: head
+        sizes of a kind they take; the window and the block mask they know, the gate is applied behind them."""
+        from ..kernels import attn_tc
+        return attn_tc.sizes_fit(self.hd, self.hdv) and not self.score_options
 
     def _fast_extended(self) -> bool:
         """Whether a layer with the further options can go to the tensor-core kernels that know them (mma.sync):
         equal head sizes of a kind they take, no block mask, no gate a head."""
-        return (self.extended and self.hdv == self.hd and self.hd % 16 == 0 and 16 <= self.hd <= 256
+        return (self.score_options and self.hdv == self.hd and self.hd % 16 == 0 and 16 <= self.hd <= 256
                 and self.block is None and not self.head_gate and self.own_kv)
 
     def bind(self, tensors, rt):

@@ -40,6 +40,7 @@ class RoutedExperts(FeedForward):
       normalise=True         the chosen outputs' weights are divided by their sum (+ 1e-20)
       weight_scale           a constant on the weights (behind the normalisation)
       score="logits"         s = z itself; the chosen outputs' weights are the softmax over the chosen logits only
+      logit_bias=True        z has a stored bias added (tensor ``router.bias``), before scores and choice (no correction then)
       expert="relu_squared"  an expert (and the shared one) is down(max(up h, 0)^2): no gate matrix
       expert="gated_clamped" an expert is down(g' sigmoid(alpha g') (u' + shift)) with g' = min(gate h, limit) and u' =
                              clamp(up h, -limit, limit); ``clamp`` = (limit, alpha, shift), and ``shared_limit`` the shared
@@ -62,12 +63,14 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, inner: int, n_experts: int, top: int, n_identity: int = 0, groups: tuple | None = None,
                  shared_inner: int | None = None, correction: bool = True, score: str = "softmax", group_score: str = "max",
                  normalise: bool = False, weight_scale: float = 1.0, expert: str = "gated_silu", clamp: tuple | None = None,
-                 shared_limit: float | None = None, shared_gate: bool = False):
+                 shared_limit: float | None = None, shared_gate: bool = False, logit_bias: bool = False):
         self.width, self.inner, self.ne, self.top = int(width), int(inner), int(n_experts), int(top)
         self.ni = int(n_identity or 0)
         self.n_out = self.ne + self.ni
         self.groups = (int(groups[0]), int(groups[1])) if groups else (1, 1)
-        self.correction = bool(correction)
+        self.correction, self.logit_bias = bool(correction), bool(logit_bias)
+        if self.correction and self.logit_bias:
+            raise ValueError("routed_experts: a bias of the logits and a correction of the choice are not built together")
         if self.top > self.n_out or self.n_out % self.groups[0] or not (1 <= self.groups[1] <= self.groups[0]):
             raise ValueError("routed_experts: top must not exceed the router's outputs, which divide into equal groups")
         if self.n_out > 1024 or self.ne < 1:
@@ -77,7 +80,7 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: score is 'softmax', 'sigmoid' or 'logits', group_score 'max' or 'top2_sum', expert "
                              "'gated_silu', 'relu_squared' or 'gated_clamped'")
         self.mode = ({"softmax": 0, "sigmoid": ops.ROUTE_SIGMOID, "logits": ops.ROUTE_LOGITS}[score] | (ops.ROUTE_GROUP_TOP2 if group_score == "top2_sum" else 0)
-                     | (ops.ROUTE_NORMALISE if normalise else 0))
+                     | (ops.ROUTE_NORMALISE if normalise else 0) | (ops.ROUTE_LOGIT_BIAS if self.logit_bias else 0))
         self.weight_scale, self.gated = float(weight_scale), expert != "relu_squared"
         if (expert == "gated_clamped") != (clamp is not None):
             raise ValueError("routed_experts: clamp = (limit, alpha, shift) goes with 'gated_clamped' experts")
@@ -102,6 +105,8 @@ class RoutedExperts(FeedForward):
         s = [W("router.weight", (self.n_out, self.width), "matrix", ("normal", 0.3))]
         if self.correction:
             s.append(W("correction", (self.n_out,), "vector", ("normal", 0.05)))
+        if self.logit_bias:
+            s.append(W("router.bias", (self.n_out,), "vector", ("normal", 0.2)))
         for e in range(self.ne):
             if self.gated:
                 s.append(W(f"experts.{e}.gate_proj.weight", (self.inner, self.width)))
@@ -130,7 +135,8 @@ class RoutedExperts(FeedForward):
             wr = torch.cat([wr, tensors["shared.out_gate.weight"].to(wr.dtype)], dim=0)
         self.w_router = wr.contiguous() if (wr.dtype == torch.bfloat16 and rt.dtype == torch.bfloat16 and self.width % 8 == 0) \
             else wr.float().contiguous()
-        self.corr = tensors["correction"].float().contiguous() if self.correction else None
+        self.corr = tensors["correction"].float().contiguous() if self.correction else \
+            tensors["router.bias"].float().contiguous() if self.logit_bias else None
         g0 = tensors["experts.0.up_proj.weight"]
         rows = 2 * self.inner if self.gated else self.inner          # [gate ; up] or up alone
         self.w_gu = torch.empty((self.ne, rows, self.width), dtype=g0.dtype, device=g0.device)
