@@ -546,6 +546,31 @@ def bozavik_config(z):
             "embedding": {"scale": 12.0}, "residual_mult": 0.3, "layers": layers}
 
 
+def demazen_config(z):
+    """Layers in fours: a matrix memory, twice windowed attention beside gated linear attention, a matrix memory; the first layer
+    with a dense feed-forward, the others routed with an active size (the chosen experts) of the dense models' ff.  Keys have
+    half the size of values in every mixer."""
+    memory = {"heads": z["width"] // 256, "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"] // 2, "vdim": z["dim"], "scale": (z["dim"] // 2) ** -0.5,
+            "mask": {"size": 1024}}
+    right = {"heads": z["heads"], "dim": z["dim"] // 2, "vdim": z["dim"], "tau": 16.0, "rank": 16}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 6}, "router": {"experts": 32, "top": 6}}
+    layers = []
+    for i in range(z["layers"]):
+        mlp = {"kind": "dense", "ff": z["ff"]} if i == 0 else dict(moe)
+        if i % 4 in (0, 3):
+            layers.append({"type": "mlstm", "mixer": dict(memory), "mlp": mlp})
+        else:
+            layers.append({"type": "parallel", "mixer": {"left": dict(left), "right": dict(right)}, "mlp": mlp})
+    return {"architecture": "Demazen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "max_positions": 8192, "layers": layers}
+
+
+def demazen_times(args):
+    return design_times(args, "demazen", (("demazen", demazen_config), ("tinuzen", tinuzen_config), ("vusalix", vusalix_config),
+                                          ("qwen3", qwen3_config_like)))
+
+
 def bozavik_times(args):
     return design_times(args, "bozavik", (("bozavik", bozavik_config), ("vusalix", vusalix_config), ("qwen3", qwen3_config_like)))
 
@@ -1000,7 +1025,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (named in config)")
     ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "timeline", "timeline-prefill", "sample", "attention", "peaks", "sugizen", "tinuzen", "vusalix",
-                             "bizepel", "bozavik"],
+                             "bizepel", "bozavik", "demazen"],
                     help="a part of the run only (for profiling); the JSON line then holds that part. "
                          "timeline: every kernel of a decode step with its begin and end inside the graph "
                          "(timeline-prefill: of a prompt); "
@@ -1011,7 +1036,8 @@ def main():
                          "tinuzen: the same for the Tinuzen design beside Sugizen and Qwen3; "
                          "vusalix: the same for the Vusalix design beside Sugizen and Qwen3; "
                          "bizepel: the same for the Bizepel design beside Vusalix, Tinuzen and Qwen3; "
-                         "bozavik: the same for the Bozavik design beside Vusalix and Qwen3")
+                         "bozavik: the same for the Bozavik design beside Vusalix and Qwen3; "
+                         "demazen: the same for the Demazen design beside Tinuzen, Vusalix and Qwen3")
     ap.add_argument("--batch", type=int, default=BATCH, help="sequences of the decode step")
     ap.add_argument("--fast-fill", action="store_true", help="do not run the prompts; mark the cache as filled")
     ap.add_argument("--prompt", type=int, default=PROMPT, help="positions each sequence holds before the timed steps")
@@ -1050,6 +1076,8 @@ def main():
         return vusalix_times(args)
     if args.only == "bizepel":
         return bizepel_times(args)
+    if args.only == "demazen":
+        return demazen_times(args)
     if args.only == "bozavik":
         return bozavik_times(args)
     if args.config != "8b":

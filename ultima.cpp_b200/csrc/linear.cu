@@ -104,7 +104,7 @@ lin_gates_kernel(const float* __restrict__ p, LinShape s, const float* __restric
     const int t0 = seq_start[b], t1 = seq_start[b + 1];
     if (t0 >= t1) return;
     float* ms = m_state + (long long)seq_slot[b] * s.H + h;
-    float m = *ms;                                            // the maximum before this round's first token
+    float m = *ms;                                            // the maximum before this turn's first token
     for (int base = t0; base < t1; base += GATE_WARPS * 32) {
         const int t = base + threadIdx.x;
         float f1 = 0.f, i1 = -INFINITY;                       // past the end: the map that changes nothing
@@ -373,7 +373,7 @@ lin_scan_kernel(ScanParams a, LinShape s) {
                 for (int tt = 0; tt < cnt; ++tt) token(tt);
             }
         }
-        __syncthreads();                                       // this buffer is asked for again in the next round
+        __syncthreads();                                       // this buffer is asked for again in the next turn
     }
     if (!busy || (PASS == SCAN_OUT && t1 != s1)) return;
 #pragma unroll
