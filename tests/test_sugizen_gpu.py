@@ -40,10 +40,11 @@ def test_norm_on_a_sublayers_output(width):
     ref = x.double() + P.rms_norm(y.double(), w.double(), 1e-5)
     xd, yd = x.to(DEV), y.to(DEV)
     h = torch.empty(5, width, dtype=torch.bfloat16, device=DEV)
-    ops.rmsnorm_add(yd, w.to(DEV), xd, 1e-5, h=h, clear_y=True)
+    after = (ops.NEXT_RMS, w.to(DEV), None, 1e-5)
+    ops.norm_join(yd, xd, 1.0, after, ops.NEXT_PLAIN, None, h)
     assert rel_err(xd, ref) < 1e-6 and rel_err(h, ref) < 2 ** -7 and float(yd.abs().max()) == 0.0
     xd, yd = x.to(DEV), y.to(DEV)
-    ops.rmsnorm_add(yd, w.to(DEV), xd, 1e-5)
+    ops.norm_join(yd, xd, 1.0, after, clear_y=False)
     assert rel_err(xd, ref) < 1e-6 and torch.equal(yd.cpu(), y)
 
 

@@ -491,45 +491,6 @@ UB_API int ub_qk_prepare(const void* qkv, int in_dtype, int n_parts, long long p
 }
 
 // ---------------------------------------------------------------------------------------
-// The norm on a sublayer's output: x[r, :] += y[r, :] * w / sqrt(mean(y[r, :]^2) + eps), x and y
-// float32.  In the same pass the kernel can hand the next sublayer its input (``h`` = the new x in the
-// activation type) and clear y, which sublayers add their output into.
-// ---------------------------------------------------------------------------------------
-template <typename TH>
-__global__ void rmsnorm_add_kernel(float* __restrict__ y, const float* __restrict__ w, float* __restrict__ x,
-                                   TH* __restrict__ h, int width, float eps, int clear_y) {
-    __shared__ float red[33];
-    pdl_trigger();
-    pdl_wait();
-    const long long r = blockIdx.x;
-    float* yr = y + r * width;
-    float* xr = x + r * width;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) { const float v = yr[i]; ss += v * v; }
-    ss = block_sum(ss, red);
-    const float inv = inv_rms(ss, (float)width, eps);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = xr[i] + yr[i] * w[i] * inv;
-        xr[i] = v;
-        if (h) h[r * width + i] = from_f32<TH>(v);
-        if (clear_y) yr[i] = 0.f;
-    }
-}
-
-UB_API int ub_rmsnorm_add(float* y, const float* w, float* x, void* h, int h_dtype, int n_rows, int width,
-                          float eps, int clear_y, cudaStream_t st) {
-    if (n_rows <= 0) return 0;
-    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
-    cudaError_t e;
-    if (h == nullptr || h_dtype == UB_F32)
-        e = ub_launch_dependent(rmsnorm_add_kernel<float>, dim3(n_rows), dim3(threads), 0, st, y, w, x, (float*)h, width, eps, clear_y);
-    else if (h_dtype == UB_BF16)
-        e = ub_launch_dependent(rmsnorm_add_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), 0, st, y, w, x, (__nv_bfloat16*)h, width, eps, clear_y);
-    else return UB_ERR_UNSUPPORTED;
-    return (int)e;
-}
-
-// ---------------------------------------------------------------------------------------
 // The clamped gate product: with g' = min(g, limit) and u' = clamp(u, -limit, limit),
 // out[t, f] = g' * sigmoid(alpha * g') * (u' + shift); gate and up side by side in one row of gu.
 // ---------------------------------------------------------------------------------------

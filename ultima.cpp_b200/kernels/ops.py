@@ -103,7 +103,6 @@ def _declare(lib, source: str) -> None:
             "ub_rotate_pairs": [P, I, L, I, I, I, P, P, P, I, I, P],
             "ub_kv_write": [P, P, I, L, P, P, P, P, I, P, I, I, I, I, I, I, P],
             "ub_silu_mul": [P, I, I, L, P, I, I, I, P],
-            "ub_rmsnorm_add": [P, P, P, P, I, I, I, F, I, P],
             "ub_glu_clamped": [P, I, P, I, I, I, F, F, F, P, L, P],
             "ub_head_gate": [P, I, L, P, L, I, I, I, P],
             "ub_convert": [P, I, P, I, L, P],
@@ -332,17 +331,6 @@ def silu_mul(gate_up, out):
     assert out.is_contiguous()
     _check(_lib("basic.cu").ub_silu_mul(_ptr(gate_up), _code(gate_up), n_parts, part_stride, _ptr(out),
                                         _code(out), T, F, _stream()), "silu_mul")
-
-
-def rmsnorm_add(y, weight, x, eps, h=None, clear_y=False):
-    """x += y * weight / sqrt(mean(y^2) + eps), row by row (x, y float32).  ``h``: the new x in h's type,
-    for the next reader; ``clear_y``: y is zeroed behind the read."""
-    _need_cuda(y, weight, x, h)
-    n, width = x.shape
-    assert x.dtype == y.dtype == weight.dtype == torch.float32 and y.shape == x.shape and weight.numel() == width
-    assert x.is_contiguous() and y.is_contiguous() and (h is None or (h.is_contiguous() and h.shape == x.shape))
-    _check(_lib("basic.cu").ub_rmsnorm_add(_ptr(y), _ptr(weight), _ptr(x), _ptr(h), _code(h) if h is not None else F32,
-                                           n, width, float(eps), 1 if clear_y else 0, _stream()), "rmsnorm_add")
 
 
 def glu_clamped(gate_up, out, limit, alpha, shift, row_gate=None):

@@ -44,6 +44,9 @@ class _NormAfter(Arrangement):
     the first.  A mixer that leaves two results (``apart``) gets a second such buffer, and its own joining kernel
     applies this norm behind its own."""
 
+    def kernel_needs(self, run_dtype):
+        return [("rowwise.cu", ())]
+
     def _buffers(self, x, rt):
         carry = getattr(rt, "_norm_after_carry", None)
         if carry is not None and carry[0] == (rt.pass_id, x.data_ptr(), tuple(x.shape)):

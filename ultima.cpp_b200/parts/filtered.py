@@ -183,7 +183,7 @@ class TokenSide(Tail):
         y = rt.arena.alloc((T, self.width), torch.float32)
         rt.matmul(g, self.w_proj, y)
         rt.launches += 1
-        ops.rmsnorm_add(y, self.norm_w, x, self.eps)
+        ops.norm_join(y, x, 1.0, (ops.NEXT_RMS, self.norm_w, None, self.eps), clear_y=False)
 
 
 class _PreNormFiltered(Arrangement):

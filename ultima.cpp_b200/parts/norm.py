@@ -33,7 +33,8 @@ class RMSNorm(Norm):
         """x += norm(y), for layers that norm a sublayer's output instead of its input; x, y float32
         [T, width].  ``h`` receives the new x in h's type (the next sublayer's input); ``clear`` zeroes y."""
         rt.launches += 1
-        ops.rmsnorm_add(y, self.weight, x, self.eps, h=h, clear_y=clear)
+        ops.norm_join(y, x, 1.0, (ops.NEXT_RMS, self.weight, None, self.eps), ops.NEXT_PLAIN if h is not None else ops.NEXT_NONE,
+                      None, h, clear_y=clear)
 
 
 @register_part("norm", "layer")
