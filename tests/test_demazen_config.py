@@ -91,6 +91,8 @@ def test_the_model_as_data():
     # what is compiled: attention once for each pair of sizes the tensor-core kernels take
     pairs = {d for s, d in spec.kernel_needs(torch.bfloat16) if s == "attn_mma.cu"}
     assert pairs == {("HEAD_DIM=32", "HEAD_DIM_V=48"), ("HEAD_DIM=16",)}
+    wide = {d for s, d in model_spec_for(u.config_from_dict(WIDE)).kernel_needs(torch.bfloat16) if s == "attn_tcgen05.cu"}
+    assert wide == {("HEAD_DIM=64", "HEAD_DIM_V=128"), ("HEAD_DIM=128",), ("HEAD_DIM=128", "HEAD_DIM_V=256")}
     assert not any(s == "attn_mma.cu" for s, _ in model_spec_for(u.config_from_dict(ODD)).kernel_needs(torch.bfloat16))
     assert not any(s == "attn_mma.cu" for s, _ in spec.kernel_needs(torch.float32))
 

@@ -412,16 +412,29 @@ def _attention_case(nh, nkv, hd, hdv, befores, news, window, seed, slices=None, 
     return worst
 
 
-TWO_SIZES = [(4, 2, 64, 128), (6, 3, 32, 48), (3, 3, 96, 16), (2, 1, 128, 256), (8, 2, 16, 32), (16, 2, 48, 112), (4, 4, 256, 64), (5, 1, 128, 64)]
+TWO_SIZES = [(4, 2, 64, 128), (6, 3, 32, 48), (3, 3, 96, 16), (2, 1, 128, 256), (8, 2, 16, 32), (16, 2, 48, 112), (4, 4, 256, 64), (5, 1, 128, 64),
+             (6, 2, 96, 192), (2, 2, 112, 96), (3, 1, 208, 224)]
 
 
+@pytest.mark.parametrize("kernel", [None, "mma", "wide"])
 @pytest.mark.parametrize("nh,nkv,hd,hdv", TWO_SIZES)
-def test_attention_of_prompts_with_values_of_another_size(nh, nkv, hd, hdv):
-    for window in (None, 40, 1, 100):
-        err = _attention_case(nh, nkv, hd, hdv, [0, 0, 0, 70], [1, 17, 130, 65], window, seed=hd + hdv)
-        assert err <= 2 ** -6, (window, err)
-    err = _attention_case(nh, nkv, hd, hdv, [0, 200], [300, 70], 150, seed=hd, ring_pages=6)      # (the second one's ring has wrapped)
-    assert err <= 2 ** -6, err
+def test_attention_of_prompts_with_values_of_another_size(nh, nkv, hd, hdv, kernel):
+    """On tcgen05 where the sizes fit (128 rows a CTA, and 256 where the values do), and on mma.sync; rows that end inside a block
+    of 64 columns, heads that do and do not divide 128, continued prompts, a ring that has wrapped."""
+    from ultima_b200.kernels import attn_tc
+    if kernel == "wide" and (not attn_tc.tc_sizes_fit(hd, hdv) or hdv > 128):
+        pytest.skip("not a size of that kernel")
+    held = attn_tc.WIDE
+    attn_tc.set_wide(2 if kernel == "wide" else 0)
+    try:
+        k = None if kernel == "wide" else kernel
+        for window in (None, 40, 1, 100):
+            err = _attention_case(nh, nkv, hd, hdv, [0, 0, 0, 70], [1, 17, 130, 65], window, seed=hd + hdv, kernel=k)
+            assert err <= 2 ** -6, (window, err)
+        err = _attention_case(nh, nkv, hd, hdv, [0, 200], [300, 70], 150, seed=hd, ring_pages=6, kernel=k)
+        assert err <= 2 ** -6, err
+    finally:
+        attn_tc.set_wide(held)
 
 
 @pytest.mark.parametrize("nh,nkv,hd,hdv", TWO_SIZES)

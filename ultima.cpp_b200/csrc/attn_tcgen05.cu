@@ -1,5 +1,7 @@
 // Attention over the paged bfloat16 cache on the fifth-generation tensor cores, for prompts and for
-// decode steps, for one head size fixed at compile time (-DHEAD_DIM=64 or 128).
+// decode steps, for one head size fixed at compile time (-DHEAD_DIM=64 or 128), and, for prompts only, for values of another
+// size than keys (-DHEAD_DIM=, a multiple of 16, and -DHEAD_DIM_V=, a multiple of 32, both up to 256; rows that end inside a
+// block of 64 columns are padded with zeros by the copies).
 //
 // One CTA takes 128 rows of one KV head, a row being (token, query head of the group), and walks
 // over the cache pages (64 keys) its rows may see.  Scores and the output live in tensor memory:
@@ -28,16 +30,25 @@
 #ifndef HEAD_DIM
 #define HEAD_DIM 128
 #endif
-static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "this kernel is built for head sizes 64 and 128");
+#ifndef HEAD_DIM_V
+#define HEAD_DIM_V HEAD_DIM
+#endif
+constexpr bool SAME = HEAD_DIM == HEAD_DIM_V;
+static_assert(SAME ? (HEAD_DIM == 64 || HEAD_DIM == 128)
+                   : (HEAD_DIM % 16 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= 256 && HEAD_DIM_V % 32 == 0 && HEAD_DIM_V >= 32 && HEAD_DIM_V <= 256),
+              "this kernel is built for head sizes 64 and 128, or for unequal sizes up to 256 (keys in sixteens, values in thirty-twos)");
 
-constexpr int HD = HEAD_DIM;
-constexpr int NB = HD / 64;                 // 64-column blocks of a row (one 128-byte swizzle span each)
+constexpr int HD = HEAD_DIM;                // queries and keys
+constexpr int HDV = HEAD_DIM_V;             // values and outputs
+constexpr int NB = (HD + 63) / 64;          // 64-column blocks of a row (one 128-byte swizzle span each)
+constexpr int NBV = (HDV + 63) / 64;
 constexpr int BM = 128;                     // rows a CTA
 constexpr int BN = 64;                      // keys a tile = positions a page
 constexpr int Q_BYTES = NB * BM * 128;
-constexpr int KV_BYTES = NB * BN * 128;     // one K or V tile
-constexpr int smem_bytes(int stages) { return Q_BYTES + 2 * stages * KV_BYTES + 1024 + 256; }
-constexpr int TMEM_COLS = 256;              // S0 [0,64) S1 [64,128) O [128, 128 + HD)
+constexpr int K_BYTES = NB * BN * 128;      // one K tile
+constexpr int V_BYTES = NBV * BN * 128;     // one V tile
+constexpr int smem_bytes(int stages) { return Q_BYTES + stages * (K_BYTES + V_BYTES) + 1024 + 256; }
+constexpr int TMEM_COLS = HDV <= 128 ? 256 : 512;       // S0 [0,64) S1 [64,128) O [128, 128 + HDV)
 constexpr int O_COL = 128;
 constexpr float RESCALE_STEP = 8.0f;        // log2 units the reference maximum may lag behind
 constexpr int NTHREADS = 192;
@@ -57,7 +68,7 @@ struct TcAttnParams {
     float* part_o; float* part_ml; int n_slices, nh;
     int n_seqs, n_row_tiles;                  // prompts: the grid is n_row_tiles * n_seqs * nkv blocks
     // prompts only: a sink in the softmax's sum (one more term exp(0) that brings no value), a constant on the
-    // output, and one gate an output element (float32 [tokens, heads * HD], row stride g_stride) whose sigmoid
+    // output, and one gate an output element (float32 [tokens, heads * HDV], row stride g_stride) whose sigmoid
     // multiplies the output
     int sink; float out_scale; const float* gate; long long g_stride;
 };
@@ -148,8 +159,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint8_t* q_s = smem;
     uint8_t* k_s = q_s + Q_BYTES;
-    uint8_t* v_s = k_s + KV_STAGES * KV_BYTES;
-    uint64_t* bars = (uint64_t*)(v_s + KV_STAGES * KV_BYTES);
+    uint8_t* v_s = k_s + KV_STAGES * K_BYTES;
+    uint64_t* bars = (uint64_t*)(v_s + KV_STAGES * V_BYTES);
     uint64_t* q_full = bars;
     uint64_t* k_full = bars + 1;
     uint64_t* k_empty = k_full + KV_STAGES;
@@ -220,8 +231,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     const int j = armed_k, s = j % KV_STAGES;
                     if (mbar_test_wait(&k_empty[s], (uint32_t)(((j / KV_STAGES) & 1) ^ 1))) {
                         const int row = row_of(j);
-                        mbar_expect_tx(&k_full[s], KV_BYTES);
-                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(k_s + s * KV_BYTES + nb * BN * 128, &map_k, &k_full[s], nb * 64, row);
+                        mbar_expect_tx(&k_full[s], K_BYTES);
+                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(k_s + s * K_BYTES + nb * BN * 128, &map_k, &k_full[s], nb * 64, row);
                         armed_k = j + 1;
                         moved = true;
                     }
@@ -230,8 +241,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     const int j = armed_v, s = j % KV_STAGES;
                     if (mbar_test_wait(&v_empty[s], (uint32_t)(((j / KV_STAGES) & 1) ^ 1))) {
                         const int row = row_of(j);
-                        mbar_expect_tx(&v_full[s], KV_BYTES);
-                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(v_s + s * KV_BYTES + nb * BN * 128, &map_v, &v_full[s], nb * 64, row);
+                        mbar_expect_tx(&v_full[s], V_BYTES);
+                        for (int nb = 0; nb < NBV; ++nb) tma_load_2d(v_s + s * V_BYTES + nb * BN * 128, &map_v, &v_full[s], nb * 64, row);
                         armed_v = j + 1;
                         moved = true;
                     }
@@ -256,13 +267,13 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             // Every descriptor is a constant away from three made once: the address field counts 16-byte
             // units and shared memory ends far below where it would carry into the next field.
             constexpr uint32_t idesc_qk = idesc_bf16(BM, BN, 0);
-            constexpr uint32_t idesc_pv = idesc_bf16(BM, HD, 1);          // all HD output columns in one MMA
+            constexpr uint32_t idesc_pv = idesc_bf16(BM, HDV, 1);         // all HDV output columns in one MMA
             const uint64_t q_desc = make_desc(smem_u32(q_s));
             const uint64_t k_desc = make_desc(smem_u32(k_s));
             const uint64_t v_desc = make_desc_mn(smem_u32(v_s));
             auto issue_qk = [&](int j) {
                 const int s = j % KV_STAGES;
-                const uint64_t kd = k_desc + (uint64_t)(s * (KV_BYTES >> 4));
+                const uint64_t kd = k_desc + (uint64_t)(s * (K_BYTES >> 4));
                 const uint32_t acc = tmem_base + (uint32_t)((j & 1) * BN);
 #pragma unroll
                 for (int ks = 0; ks < HD / 16; ++ks) {
@@ -289,7 +300,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 if (ok) ok = mbar_wait(&v_full[j % KV_STAGES], (uint32_t)((j / KV_STAGES) & 1), err);
                 if (!ok) break;
                 tc_fence_after();
-                const uint64_t vd = v_desc + (uint64_t)((j % KV_STAGES) * (KV_BYTES >> 4));
+                const uint64_t vd = v_desc + (uint64_t)((j % KV_STAGES) * (V_BYTES >> 4));
                 const uint32_t p_t = tmem_base + (uint32_t)((j & 1) * BN);
 #pragma unroll
                 for (int ks = 0; ks < BN / 16; ++ks)
@@ -319,9 +330,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 ok = mbar_wait(&v_full[j % KV_STAGES], (uint32_t)((j / KV_STAGES) & 1), err);
                 if (!ok) break;
                 const int first = last_pos + 1 - base;     // first row to clear (>= 1: the tile holds a valid key)
-                uint8_t* vt = v_s + (j % KV_STAGES) * KV_BYTES;
-                for (int i = st; i < (BN - first) * NB * 8; i += 128) {
-                    const int row = first + i / (NB * 8), rest = i % (NB * 8);
+                uint8_t* vt = v_s + (j % KV_STAGES) * V_BYTES;
+                for (int i = st; i < (BN - first) * NBV * 8; i += 128) {
+                    const int row = first + i / (NBV * 8), rest = i % (NBV * 8);
                     *reinterpret_cast<uint4*>(vt + (rest / 8) * BN * 128 + row * 128 + (rest % 8) * 16) = make_uint4(0, 0, 0, 0);
                 }
                 fence_proxy_async();
@@ -363,7 +374,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     if (!ok) break;
                     tc_fence_after();
 #pragma unroll
-                    for (int cb = 0; cb < HD / 32; ++cb) {
+                    for (int cb = 0; cb < HDV / 32; ++cb) {
                         uint32_t oo[32];
                         tmem_ld32(lane_addr + (uint32_t)(O_COL + cb * 32), oo);
                         tmem_ld_wait();
@@ -405,12 +416,12 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             const bool partial = DECODE && p.n_slices > 1;
             const float inv = partial ? 1.0f : (l > 0.f ? p.out_scale / l : 0.f);
             const int head = kvh * G + g;
-            bf16* dst = p.out + (long long)(q0 + tok) * p.o_stride + (long long)head * HD;
-            const float* gt = (!DECODE && p.gate && row_ok) ? p.gate + (long long)(q0 + tok) * p.g_stride + (long long)head * HD : nullptr;
+            bf16* dst = p.out + (long long)(q0 + tok) * p.o_stride + (long long)head * HDV;
+            const float* gt = (!DECODE && p.gate && row_ok) ? p.gate + (long long)(q0 + tok) * p.g_stride + (long long)head * HDV : nullptr;
             const long long pi = partial ? ((long long)seq * p.nh + head) * p.n_slices + blockIdx.x : 0;
             if (partial && row_ok) { p.part_ml[pi * 2] = m_ref; p.part_ml[pi * 2 + 1] = l; }
 #pragma unroll
-            for (int cb = 0; cb < HD / 32; ++cb) {
+            for (int cb = 0; cb < HDV / 32; ++cb) {
                 uint32_t oo[32];
                 if (n_tiles > 0) {
                     tmem_ld32(lane_addr + (uint32_t)(O_COL + cb * 32), oo);
@@ -422,7 +433,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 if (row_ok && partial) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 4)
-                        *reinterpret_cast<uint4*>(p.part_o + pi * HD + cb * 32 + i) = make_uint4(oo[i], oo[i + 1], oo[i + 2], oo[i + 3]);
+                        *reinterpret_cast<uint4*>(p.part_o + pi * HDV + cb * 32 + i) = make_uint4(oo[i], oo[i + 1], oo[i + 2], oo[i + 3]);
                 } else if (row_ok) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 8)
@@ -450,12 +461,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 // into), warps 4-7 and 8-11 are the two tiles' softmax.  A key tile's place is given back when both
 // issuers have let go of it; an issuer whose rows do not see a tile lets go of it at once.
 constexpr int WIDE_TILES = 2;
-constexpr int WIDE_STAGES = HD == 128 ? 4 : 8;
+// (values of up to 128 only: both tiles' outputs share the tensor memory with four score buffers)
+constexpr int WIDE_STAGES_FIT = (220 * 1024 - WIDE_TILES * Q_BYTES) / (K_BYTES + V_BYTES);
+constexpr int WIDE_STAGES = SAME ? (HD == 128 ? 4 : 8) : WIDE_STAGES_FIT > 8 ? 8 : WIDE_STAGES_FIT < 1 ? 1 : WIDE_STAGES_FIT;
+constexpr bool WIDE_FITS = HDV <= 128 && WIDE_STAGES_FIT >= 3;
 constexpr int WIDE_THREADS = 384;
 constexpr int WIDE_TMEM = 512;
 constexpr int WIDE_O_COL = 256;
 constexpr int WIDE_MIN_BLOCKS = 148;         // fewer blocks than SMs: the kernel of 128 rows a CTA spreads the work further
-constexpr int wide_smem_bytes() { return WIDE_TILES * Q_BYTES + 2 * WIDE_STAGES * KV_BYTES + 1024 + 512; }
+constexpr int wide_smem_bytes() { return WIDE_TILES * Q_BYTES + WIDE_STAGES * (K_BYTES + V_BYTES) + 1024 + 512; }
 
 __global__ void __launch_bounds__(WIDE_THREADS, 1)
 attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -475,8 +489,8 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     uint8_t* q_s = smem;
     uint8_t* k_s = q_s + WIDE_TILES * Q_BYTES;
-    uint8_t* v_s = k_s + S * KV_BYTES;
-    uint64_t* bars = (uint64_t*)(v_s + S * KV_BYTES);
+    uint8_t* v_s = k_s + S * K_BYTES;
+    uint64_t* bars = (uint64_t*)(v_s + S * V_BYTES);
     uint64_t* q_full = bars;                               // [2]
     uint64_t* k_full = q_full + WIDE_TILES;
     uint64_t* k_empty = k_full + S;
@@ -549,8 +563,8 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     const int j = armed_k, s = j % S;
                     if (mbar_test_wait(&k_empty[s], (uint32_t)(((j / S) & 1) ^ 1))) {
                         const int row = row_of(j);
-                        mbar_expect_tx(&k_full[s], KV_BYTES);
-                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(k_s + s * KV_BYTES + nb * BN * 128, &map_k, &k_full[s], nb * 64, row);
+                        mbar_expect_tx(&k_full[s], K_BYTES);
+                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(k_s + s * K_BYTES + nb * BN * 128, &map_k, &k_full[s], nb * 64, row);
                         armed_k = j + 1;
                         moved = true;
                     }
@@ -559,8 +573,8 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     const int j = armed_v, s = j % S;
                     if (mbar_test_wait(&v_empty[s], (uint32_t)(((j / S) & 1) ^ 1))) {
                         const int row = row_of(j);
-                        mbar_expect_tx(&v_full[s], KV_BYTES);
-                        for (int nb = 0; nb < NB; ++nb) tma_load_2d(v_s + s * KV_BYTES + nb * BN * 128, &map_v, &v_full[s], nb * 64, row);
+                        mbar_expect_tx(&v_full[s], V_BYTES);
+                        for (int nb = 0; nb < NBV; ++nb) tma_load_2d(v_s + s * V_BYTES + nb * BN * 128, &map_v, &v_full[s], nb * 64, row);
                         armed_v = j + 1;
                         moved = true;
                     }
@@ -587,12 +601,12 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             const int first = has[t] ? lo[t] - t_lo : 0;
             const int n_act = has[t] ? hi[t] - lo[t] + 1 : 0;
             constexpr uint32_t idesc_qk = idesc_bf16(BM, BN, 0);
-            constexpr uint32_t idesc_pv = idesc_bf16(BM, HD, 1);
+            constexpr uint32_t idesc_pv = idesc_bf16(BM, HDV, 1);
             const uint64_t q_desc = make_desc(smem_u32(q_s + t * Q_BYTES));
             const uint64_t k_desc = make_desc(smem_u32(k_s));
             const uint64_t v_desc = make_desc_mn(smem_u32(v_s));
             const uint32_t s_base = tmem_base + (uint32_t)(t * 2 * BN);
-            const uint32_t o_base = tmem_base + (uint32_t)(WIDE_O_COL + t * HD);
+            const uint32_t o_base = tmem_base + (uint32_t)(WIDE_O_COL + t * HDV);
             uint64_t* sf = s_full + 2 * t;
             uint64_t* pf = p_full + 2 * t;
             uint64_t* pd = pv_done + 2 * t;
@@ -611,7 +625,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             };
             auto issue_qk = [&](int i) {                   // i counts this tile's own key tiles
                 const int j = first + i, s = j % S;
-                const uint64_t kd = k_desc + (uint64_t)(s * (KV_BYTES >> 4));
+                const uint64_t kd = k_desc + (uint64_t)(s * (K_BYTES >> 4));
                 const uint32_t acc = s_base + (uint32_t)((i & 1) * BN);
 #pragma unroll
                 for (int ks = 0; ks < HD / 16; ++ks) {
@@ -638,7 +652,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 if (ok) ok = mbar_wait(&v_full[j % S], (uint32_t)((j / S) & 1), err);
                 if (!ok) break;
                 tc_fence_after();
-                const uint64_t vd = v_desc + (uint64_t)((j % S) * (KV_BYTES >> 4));
+                const uint64_t vd = v_desc + (uint64_t)((j % S) * (V_BYTES >> 4));
                 const uint32_t p_t = s_base + (uint32_t)((i & 1) * BN);
 #pragma unroll
                 for (int ks = 0; ks < BN / 16; ++ks)
@@ -660,7 +674,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int n_act = has[t] ? hi[t] - lo[t] + 1 : 0;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16);
         const uint32_t s_base = lane_addr + (uint32_t)(t * 2 * BN);
-        const uint32_t o_base = lane_addr + (uint32_t)(WIDE_O_COL + t * HD);
+        const uint32_t o_base = lane_addr + (uint32_t)(WIDE_O_COL + t * HDV);
         uint64_t* sf = s_full + 2 * t;
         uint64_t* pf = p_full + 2 * t;
         uint64_t* pd = pv_done + 2 * t;
@@ -678,9 +692,9 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 ok = mbar_wait(&v_full[j % S], (uint32_t)((j / S) & 1), err);
                 if (!ok) break;
                 const int zfirst = last_pos + 1 - base;    // first row to clear (>= 1: the tile holds a valid key)
-                uint8_t* vt = v_s + (j % S) * KV_BYTES;
-                for (int x = st; x < (BN - zfirst) * NB * 8; x += 128) {
-                    const int row = zfirst + x / (NB * 8), rest = x % (NB * 8);
+                uint8_t* vt = v_s + (j % S) * V_BYTES;
+                for (int x = st; x < (BN - zfirst) * NBV * 8; x += 128) {
+                    const int row = zfirst + x / (NBV * 8), rest = x % (NBV * 8);
                     *reinterpret_cast<uint4*>(vt + (rest / 8) * BN * 128 + row * 128 + (rest % 8) * 16) = make_uint4(0, 0, 0, 0);
                 }
                 fence_proxy_async();
@@ -719,7 +733,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     if (!ok) break;
                     tc_fence_after();
 #pragma unroll
-                    for (int cb = 0; cb < HD / 32; ++cb) {
+                    for (int cb = 0; cb < HDV / 32; ++cb) {
                         uint32_t oo[32];
                         tmem_ld32(o_base + (uint32_t)(cb * 32), oo);
                         tmem_ld_wait();
@@ -760,10 +774,10 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             tc_fence_after();
             const float inv = l > 0.f ? p.out_scale / l : 0.f;
             const int head = kvh * G + g;
-            bf16* dst = p.out + (long long)(q0 + tok) * p.o_stride + (long long)head * HD;
-            const float* gt = (p.gate && row_ok) ? p.gate + (long long)(q0 + tok) * p.g_stride + (long long)head * HD : nullptr;
+            bf16* dst = p.out + (long long)(q0 + tok) * p.o_stride + (long long)head * HDV;
+            const float* gt = (p.gate && row_ok) ? p.gate + (long long)(q0 + tok) * p.g_stride + (long long)head * HDV : nullptr;
 #pragma unroll
-            for (int cb = 0; cb < HD / 32; ++cb) {
+            for (int cb = 0; cb < HDV / 32; ++cb) {
                 uint32_t oo[32];
                 tmem_ld32(o_base + (uint32_t)(cb * 32), oo);
                 tmem_ld_wait();
@@ -786,6 +800,7 @@ attn_tc_wide_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 
 // ---------------------------------------------------------------------------------------
 UB_API int ub_attn_tc_head_dim() { return HD; }
+UB_API int ub_attn_tc_value_dim() { return HDV; }
 
 // tensor map of q as [tokens, heads, HD] (row stride q_stride elements), boxes of 64 x group x floor(128/group)
 UB_API int ub_attn_tc_map_q(void* out_map, const void* q, long long n_tokens, int nh, long long q_stride, int group) {
@@ -801,13 +816,13 @@ UB_API int ub_attn_tc_map_q(void* out_map, const void* q, long long n_tokens, in
                      CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? 0 : UB_ERR_ARG;
 }
-// tensor map of one run's K or V cache [pages, kv heads, 64, HD] as rows of HD, boxes of 64 x 64
-UB_API int ub_attn_tc_map_kv(void* out_map, const void* cache, long long n_pages, int nkv) {
+// tensor map of one run's K or V cache [pages, kv heads, 64, width] as rows of ``width``, boxes of 64 x 64
+UB_API int ub_attn_tc_map_kv(void* out_map, const void* cache, long long n_pages, int nkv, int width) {
     EncodeTiledFn enc = tensor_map_encoder();
     if (!enc) return UB_ERR_UNSUPPORTED;
-    if (((uintptr_t)cache & 15) || n_pages < 1) return UB_ERR_ARG;
-    cuuint64_t dims[2] = {(cuuint64_t)HD, (cuuint64_t)(n_pages * nkv * BN)};
-    cuuint64_t strides[1] = {(cuuint64_t)HD * 2};
+    if (((uintptr_t)cache & 15) || n_pages < 1 || (width != HD && width != HDV)) return UB_ERR_ARG;
+    cuuint64_t dims[2] = {(cuuint64_t)width, (cuuint64_t)(n_pages * nkv * BN)};
+    cuuint64_t strides[1] = {(cuuint64_t)width * 2};
     cuuint32_t box[2] = {64, (cuuint32_t)BN};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = enc((CUtensorMap*)out_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void*)cache, dims, strides, box, estr,
@@ -830,9 +845,9 @@ __global__ void attn_tc_combine_kernel(TcAttnParams p) {
         const float ms = p.part_ml[(base + s) * 2];
         const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
         ll += f * p.part_ml[(base + s) * 2 + 1];
-        acc += f * p.part_o[(base + s) * HD + d];
+        acc += f * p.part_o[(base + s) * HDV + d];
     }
-    p.out[(long long)p.seq_start[seq] * p.o_stride + (long long)head * HD + d] = __float2bfloat16_rn(acc / ll);
+    p.out[(long long)p.seq_start[seq] * p.o_stride + (long long)head * HDV + d] = __float2bfloat16_rn(acc / ll);
 }
 
 template <int STAGES, bool DECODE>
@@ -865,7 +880,7 @@ static int launch_wide(unsigned blocks, const void* map_q, const void* map_k, co
 }
 
 // mode 0: prompts (any numbers of new tokens); mode 1: one new token a sequence, keys in n_slices slices
-// (part_o: float32 [n_seqs, nh, n_slices, HD], part_ml: [.., 2] when n_slices > 1).
+// (part_o: float32 [n_seqs, nh, n_slices, HDV], part_ml: [.., 2] when n_slices > 1).
 static int attn_tc_launch(int mode, const void* map_q, const void* map_k, const void* map_v, void* out, long long o_stride,
                           const int* seq_start, const int* seq_before, const int* table, int pages_per_seq,
                           int ring, int page, int n_seqs, int max_new, int nh, int nkv, int window, float scale,
@@ -914,7 +929,7 @@ static int attn_tc_launch(int mode, const void* map_q, const void* map_k, const 
         p.n_seqs = n_seqs;
         const long long wide_tiles = (max_new + WIDE_TILES * tpb - 1) / (WIDE_TILES * tpb);
         const long long wide_blocks = wide_tiles * n_seqs * nkv;
-        if ((g_wide == 2 || (g_wide == 1 && wide_blocks >= WIDE_MIN_BLOCKS)) && wide_blocks <= 0x7fffffffll) {
+        if (WIDE_FITS && (g_wide == 2 || (g_wide == 1 && wide_blocks >= WIDE_MIN_BLOCKS)) && wide_blocks <= 0x7fffffffll) {
             p.n_row_tiles = (int)wide_tiles;
             return launch_wide((unsigned)wide_blocks, map_q, map_k, map_v, p, st);
         }
@@ -925,8 +940,11 @@ static int attn_tc_launch(int mode, const void* map_q, const void* map_k, const 
     }
     if (max_new != 1) return UB_ERR_ARG;
     if (p.n_slices > 1 && (!part_o || !part_ml || ((uintptr_t)part_o & 15))) return UB_ERR_ARG;
-    int rc = launch_attn<DECODE_STAGES, true>(dim3(p.n_slices, n_seqs, nkv), map_q, map_k, map_v, p, st);
-    if (rc != 0 || p.n_slices == 1) return rc;
-    cudaError_t e = ub_launch_dependent(attn_tc_combine_kernel, dim3(n_seqs * nh), dim3(HD), 0, st, p);
-    return (int)e;
+    if constexpr (SAME) {
+        int rc = launch_attn<DECODE_STAGES, true>(dim3(p.n_slices, n_seqs, nkv), map_q, map_k, map_v, p, st);
+        if (rc != 0 || p.n_slices == 1) return rc;
+        cudaError_t e = ub_launch_dependent(attn_tc_combine_kernel, dim3(n_seqs * nh), dim3(HDV), 0, st, p);
+        return (int)e;
+    }
+    return UB_ERR_UNSUPPORTED;
 }

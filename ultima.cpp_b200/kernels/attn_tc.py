@@ -72,17 +72,27 @@ USE_TMA_DECODE = _os.environ.get("ULTIMA_ATTN_TMA_DECODE", "1") != "0"
 WIDE = int(_os.environ.get("ULTIMA_ATTN_WIDE", "1"))
 
 
-def tc_target(head_dim: int):
-    return (TC_SOURCE, (f"HEAD_DIM={int(head_dim)}",))
+def tc_target(head_dim: int, value_dim: int | None = None):
+    own = (f"HEAD_DIM_V={int(value_dim)}",) if value_dim is not None and value_dim != head_dim else ()
+    return (TC_SOURCE, (f"HEAD_DIM={int(head_dim)}",) + own)
 
 
-def tc_lib(head_dim: int):
-    L = _tc_libs.get(head_dim)
+def tc_sizes_fit(head_dim: int, value_dim: int) -> bool:
+    """The sizes the tcgen05 kernels are built for: 64 and 128, and for prompts values of another size than keys (keys in
+    sixteens, values in thirty-twos, up to 256)."""
+    if head_dim == value_dim:
+        return head_dim in (64, 128)
+    return head_dim % 16 == 0 and 16 <= head_dim <= 256 and value_dim % 32 == 0 and 32 <= value_dim <= 256
+
+
+def tc_lib(head_dim: int, value_dim: int | None = None):
+    value_dim = value_dim or head_dim
+    L = _tc_libs.get((head_dim, value_dim))
     if L is None:
-        L = build.load(*tc_target(head_dim))
+        L = build.load(*tc_target(head_dim, value_dim))
         L.ub_attn_tc_map_q.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_longlong, c_int]
         L.ub_attn_tc_map_q.restype = c_int
-        L.ub_attn_tc_map_kv.argtypes = [c_void_p, c_void_p, c_longlong, c_int]
+        L.ub_attn_tc_map_kv.argtypes = [c_void_p, c_void_p, c_longlong, c_int, c_int]
         L.ub_attn_tc_map_kv.restype = c_int
         L.ub_attn_tc.argtypes = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
@@ -95,7 +105,10 @@ def tc_lib(head_dim: int):
         L.ub_attn_tc_set_wide.argtypes = [c_int]
         L.ub_attn_tc_set_wide.restype = None
         L.ub_attn_tc_set_wide(WIDE)
-        _tc_libs[head_dim] = L
+        if L.ub_attn_tc_head_dim() != head_dim or L.ub_attn_tc_value_dim() != value_dim:
+            raise KernelError(f"attention library was built for head size {L.ub_attn_tc_head_dim()} (values {L.ub_attn_tc_value_dim()}), "
+                              f"not {head_dim} ({value_dim})")
+        _tc_libs[(head_dim, value_dim)] = L
     return L
 
 
@@ -107,9 +120,9 @@ def set_wide(mode: int) -> None:
         L.ub_attn_tc_set_wide(WIDE)
 
 
-def tcgen05_fits(head_dim: int, n_heads: int, n_kv_heads: int) -> bool:
-    """The tcgen05 kernel: head sizes 64 and 128, groups of up to 128 query heads a KV head."""
-    return USE_TCGEN05 and head_dim in (64, 128) and n_heads // n_kv_heads <= 128
+def tcgen05_fits(head_dim: int, n_heads: int, n_kv_heads: int, value_dim: int | None = None) -> bool:
+    """The tcgen05 kernel: sizes it is built for, groups of up to 128 query heads a KV head."""
+    return USE_TCGEN05 and tc_sizes_fit(head_dim, value_dim or head_dim) and n_heads // n_kv_heads <= 128
 
 
 def _tc_map(key, make):
@@ -130,18 +143,19 @@ def _tc_map(key, make):
 
 def run_tcgen05(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, decode: bool, n_slices: int = 1,
                 mask: int | None = None):
-    L = tc_lib(head_dim)
+    value_dim = kv.v.shape[-1]
+    L = tc_lib(head_dim, value_dim)
     group = n_heads // n_kv_heads
     T = q.shape[0]
     mq = _tc_map(("q", q.data_ptr(), T, n_heads, q.stride(0), group, head_dim),
                  lambda a: L.ub_attn_tc_map_q(a, q.data_ptr(), T, n_heads, q.stride(0), group))
     mk = _tc_map(("kv", kv.k.data_ptr(), kv.k.shape[0], n_kv_heads, head_dim),
-                 lambda a: L.ub_attn_tc_map_kv(a, kv.k.data_ptr(), kv.k.shape[0], n_kv_heads))
-    mv = _tc_map(("kv", kv.v.data_ptr(), kv.v.shape[0], n_kv_heads, head_dim),
-                 lambda a: L.ub_attn_tc_map_kv(a, kv.v.data_ptr(), kv.v.shape[0], n_kv_heads))
+                 lambda a: L.ub_attn_tc_map_kv(a, kv.k.data_ptr(), kv.k.shape[0], n_kv_heads, head_dim))
+    mv = _tc_map(("kv", kv.v.data_ptr(), kv.v.shape[0], n_kv_heads, value_dim),
+                 lambda a: L.ub_attn_tc_map_kv(a, kv.v.data_ptr(), kv.v.shape[0], n_kv_heads, value_dim))
     part_o = part_ml = None
     if decode and n_slices > 1:
-        part_o = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, head_dim), torch.float32)
+        part_o = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, value_dim), torch.float32)
         part_ml = rt.arena.alloc((batch.n_seqs, n_heads, n_slices, 2), torch.float32)
     rc = L.ub_attn_tc(1 if decode else 0, mq, mk, mv, _ptr(out), out.stride(0), _ptr(batch.seq_start),
                       _ptr(batch.seq_before), _ptr(kv.table), kv.table.shape[1], kv.ring, kv.page, batch.n_seqs,
@@ -313,22 +327,22 @@ def attention(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, slice
               kernel: str | None = None, block: int | None = None):
     """kernel: None picks (tcgen05 for prompts where it fits, mma.sync otherwise); "mma" forces the latter.
     ``block``: mask by blocks of this many positions instead of by the cache's window.  Values may have another size than
-    keys (the mma.sync kernels then)."""
+    keys: prompts on tcgen05 where the sizes fit, single tokens on mma.sync."""
     value_dim = kv.v.shape[-1]
     same = value_dim == head_dim
-    L = lib(head_dim, value_dim)
     mask = _mask_arg(kv, block)
     reach = block or kv.window                       # how far back a token looks at most (None: to the start)
     assert out.dtype == torch.bfloat16 and out.stride(1) == 1
     group = n_heads // n_kv_heads
     decode = batch.max_new == 1 and group <= 16
-    tc_ok = (same and kernel != "mma" and tcgen05_fits(head_dim, n_heads, n_kv_heads) and out.stride(0) % 8 == 0
+    tc_ok = (kernel != "mma" and tcgen05_fits(head_dim, n_heads, n_kv_heads, value_dim) and scale > 0 and out.stride(0) % 8 == 0
              and out.data_ptr() % 16 == 0 and kv.k.is_contiguous() and kv.v.is_contiguous())
     if tc_ok and not decode:
         return run_tcgen05(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, False, mask=mask)
-    if tc_ok and decode and (USE_TCGEN05_DECODE or kernel == "tc"):
+    if tc_ok and same and decode and (USE_TCGEN05_DECODE or kernel == "tc"):
         n = slices or decode_slices(batch.n_seqs, n_kv_heads, batch.max_after, reach, per_sm=1)
         return run_tcgen05(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, True, n, mask=mask)
+    L = lib(head_dim, value_dim)
     part_o = part_ml = None
     n_slices = 1
     tma = (same and decode and head_dim % 64 == 0 and kernel in (None, "tma") and (USE_TMA_DECODE or kernel == "tma")
@@ -383,9 +397,9 @@ def attention_ext(q, kv, out, batch, n_heads, n_kv_heads, head_dim, scale, rt, w
         mq = _tc_map(("q", q.data_ptr(), T, n_heads, q.stride(0), group, head_dim),
                      lambda a: L.ub_attn_tc_map_q(a, q.data_ptr(), T, n_heads, q.stride(0), group))
         mk = _tc_map(("kv", kv.k.data_ptr(), kv.k.shape[0], n_kv_heads, head_dim),
-                     lambda a: L.ub_attn_tc_map_kv(a, kv.k.data_ptr(), kv.k.shape[0], n_kv_heads))
+                     lambda a: L.ub_attn_tc_map_kv(a, kv.k.data_ptr(), kv.k.shape[0], n_kv_heads, head_dim))
         mv = _tc_map(("kv", kv.v.data_ptr(), kv.v.shape[0], n_kv_heads, head_dim),
-                     lambda a: L.ub_attn_tc_map_kv(a, kv.v.data_ptr(), kv.v.shape[0], n_kv_heads))
+                     lambda a: L.ub_attn_tc_map_kv(a, kv.v.data_ptr(), kv.v.shape[0], n_kv_heads, head_dim))
         rc = L.ub_attn_tc_ext(mq, mk, mv, _ptr(out), out.stride(0), _ptr(batch.seq_start), _ptr(batch.seq_before),
                               _ptr(kv.table), kv.table.shape[1], kv.ring, kv.page, batch.n_seqs, batch.max_new, n_heads,
                               n_kv_heads, 0, float(scale), _ptr(rt.status[1:2]), 1 if sink else 0, float(out_scale),

@@ -188,8 +188,8 @@ class Attention(Mixer):
                 return out
             if self._fast_attention() and attn_tc.BLOCK_MASK:
                 out.append(attn_tc.target(self.hd, self.hdv))
-                if self.hd in catalog.TC_HEAD_DIMS and self.hdv == self.hd:
-                    out.append(attn_tc.tc_target(self.hd))
+                if attn_tc.tc_sizes_fit(self.hd, self.hdv):
+                    out.append(attn_tc.tc_target(self.hd, self.hdv))
             return out
         if self.hd % 16 == 0 and 16 <= self.hd <= 256:
             out = [attn_tc.target(self.hd)]
