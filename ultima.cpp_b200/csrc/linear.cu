@@ -86,10 +86,9 @@ lin_decay_kernel(const float* __restrict__ p, LinShape s, const float* __restric
 // ---------------------------------------------------------------------------------------
 constexpr int GATE_WARPS = 16;
 
-__device__ __forceinline__ void log_gates(const float* __restrict__ p, const LinShape& s, long long t, int h,
-                                          const float* __restrict__ bi, const float* __restrict__ bf, float cap, float& i, float& f) {
-    i = cap * tanhf((lin_at(p, s, t, s.x_off + h) + bi[h]) / cap);
-    f = log_sigmoid_(cap * tanhf((lin_at(p, s, t, s.y_off + h) + bf[h]) / cap));
+__device__ __forceinline__ void log_gates(float zi, float zf, float cap, float& i, float& f) {
+    i = cap * tanhf(zi / cap);
+    f = log_sigmoid_(cap * tanhf(zf / cap));
 }
 
 __global__ void __launch_bounds__(GATE_WARPS * 32)
@@ -108,7 +107,7 @@ lin_gates_kernel(const float* __restrict__ p, LinShape s, const float* __restric
     for (int base = t0; base < t1; base += GATE_WARPS * 32) {
         const int t = base + threadIdx.x;
         float f1 = 0.f, i1 = -INFINITY;                       // past the end: the map that changes nothing
-        if (t < t1) log_gates(p, s, t, h, bi, bf, cap, i1, f1);
+        if (t < t1) log_gates(lin_at(p, s, t, s.x_off + h) + bi[h], lin_at(p, s, t, s.y_off + h) + bf[h], cap, i1, f1);
         float f = f1, i = i1;                                 // the map of this warp's tokens up to and with this lane's
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -163,16 +162,37 @@ __device__ __forceinline__ uint64_t mul_pair(uint64_t a, uint64_t b) {
     return d;
 }
 
-constexpr int SCAN_LANES = 8;                 // lanes that share a column of S; each holds R of its D channels
-
-template <int R, int C, bool HEAD>
+// LANES lanes share a column of S, each with R of its D channels; a thread holds C neighbouring columns, which share its reads
+// of the token's q, k and decays (those reads and the arithmetic are about equally dear).
+template <int LANES, int R, int C, bool HEAD>
 struct ScanLayout {
-    static constexpr int DP = SCAN_LANES * R, COLS = 128 / SCAN_LANES * C;
+    static constexpr int DP = LANES * R, COLS = 128 / LANES * C;
     static constexpr int TT = DP <= 128 ? 8 : 4;              // tokens a stage
-    static constexpr int STAGES = 2;
+    static constexpr int STAGES = 3;
+    static constexpr int BLOCKS = R <= 4 ? 4 : 3;             // blocks an SM the registers are cut for
     static constexpr int TOKEN = (HEAD ? 2 : 3) * DP + COLS + 4;      // floats of a token: q, k, (decays), v, (keep, put)
     static constexpr size_t BYTES = (size_t)STAGES * TT * TOKEN * sizeof(float);
 };
+
+// The sum over a column's LANES lanes of C values each: every exchange halves the values a lane is left with, so a lane ends
+// with the sum of value ``sum_of``.
+template <int LANES, int C>
+__device__ __forceinline__ float lane_sums(float (&o)[C], int l) {
+    int mask = LANES / 2;
+#pragma unroll
+    for (int n = C / 2; n >= 1; n >>= 1, mask >>= 1) {
+        const bool up = l & mask;
+#pragma unroll
+        for (int x = 0; x < n; ++x) {
+            const float mine = up ? o[x + n] : o[x], other = up ? o[x] : o[x + n];
+            o[x] = mine + __shfl_xor_sync(0xffffffffu, other, mask);
+        }
+    }
+    float r = o[0];
+#pragma unroll
+    for (; mask >= 1; mask >>= 1) r += __shfl_xor_sync(0xffffffffu, r, mask);
+    return r;
+}
 
 struct ScanParams {
     const float* p;
@@ -191,24 +211,24 @@ enum { SCAN_WHOLE = 0, SCAN_SUM = 1, SCAN_OUT = 2 };
 // Grid (blocks of columns, heads, sequences * chunks), 128 threads.  SCAN_WHOLE: one chunk, from the slot's state to the slot's
 // state.  SCAN_SUM: from zero, no output; leaves the chunk's contribution and its total decay.  SCAN_OUT: from the state
 // before the chunk (work); the last chunk leaves the slot's state.
-// A thread holds C neighbouring columns of S and of each the channels of the float4 chunks l, l + 8, ... (l its lane in the
-// column's eight): the lanes read consecutive bytes of shared memory, and all columns of a warp the same ones.  Tokens come
-// through shared memory a stage at a time, the next stage on its way while one is worked on.
-template <int R, int C, bool HEAD, bool VEC, int PASS>
-__global__ void __launch_bounds__(128)
+// A thread holds C neighbouring columns of S and of each the channels of the float4 chunks l, l + LANES, ... (l its lane among the
+// column's): the lanes read consecutive bytes of shared memory, and all columns of a warp the same ones.  Tokens come
+// through shared memory a stage at a time, the next stages on their way while one is worked on.
+template <int LANES, int R, int C, bool HEAD, bool VEC, int PASS>
+__global__ void __launch_bounds__(128, (ScanLayout<LANES, R, C, HEAD>::BLOCKS))
 lin_scan_kernel(ScanParams a, LinShape s) {
-    using L = ScanLayout<R, C, HEAD>;
-    constexpr int DP = L::DP, COLS = L::COLS, TT = L::TT, NC = R / 4;
+    using L = ScanLayout<LANES, R, C, HEAD>;
+    constexpr int DP = L::DP, COLS = L::COLS, TT = L::TT, NC = R / 4, ST = L::STAGES;
     extern __shared__ __align__(16) float sm[];
-    float* sq = sm;                                            // [2][TT][DP]
-    float* sk = sq + 2 * TT * DP;
-    float* sa = sk + 2 * TT * DP;                              // (channel form)
-    float* sv = sa + (HEAD ? 0 : 2 * TT * DP);                 // [2][TT][COLS]
-    float* sg = sv + 2 * TT * COLS;                            // [2][TT][4]: keep, put (head form)
+    float* sq = sm;                                            // [ST][TT][DP]
+    float* sk = sq + ST * TT * DP;
+    float* sa = sk + ST * TT * DP;                             // (channel form)
+    float* sv = sa + (HEAD ? 0 : ST * TT * DP);                // [ST][TT][COLS]
+    float* sg = sv + ST * TT * COLS;                           // [ST][TT][4]: keep, put (head form)
     pdl_trigger();
     pdl_wait();
-    const int tid = threadIdx.x, l = tid % SCAN_LANES, warp = tid >> 5;
-    const int col = tid / SCAN_LANES * C;                      // the first of this thread's columns in the block
+    const int tid = threadIdx.x, l = tid % LANES, warp = tid >> 5;
+    const int col = tid / LANES * C;                      // the first of this thread's columns in the block
     const int h = blockIdx.y, b = blockIdx.z % a.n_seqs, ck = blockIdx.z / a.n_seqs;
     const int D = s.D, E = s.E, EW = a.EW, H = s.H;
     const int j0 = blockIdx.x * COLS, j = j0 + col;
@@ -230,7 +250,7 @@ lin_scan_kernel(ScanParams a, LinShape s) {
     for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
-            const int d = (c * SCAN_LANES + l) * 4 + 2 * u;
+            const int d = (c * LANES + l) * 4 + 2 * u;
 #pragma unroll
             for (int x = 0; x < C; ++x) {
                 float v0 = 0.f, v1 = 0.f;
@@ -242,15 +262,16 @@ lin_scan_kernel(ScanParams a, LinShape s) {
             }
         }
     // channels and columns past the sizes are constants that no copy ever touches; the column behind the values is 1
-    for (int i = tid; i < 2 * TT * DP; i += blockDim.x)
+    for (int i = tid; i < ST * TT * DP; i += blockDim.x)
         if (i % DP >= D) { sq[i] = 0.f; sk[i] = 0.f; if (!HEAD) sa[i] = 1.f; }
-    for (int i = tid; i < 2 * TT * COLS; i += blockDim.x) {
+    for (int i = tid; i < ST * TT * COLS; i += blockDim.x) {
         const int jj = j0 + i % COLS;
         if (jj >= E) sv[i] = (jj == E && EW > E) ? 1.f : 0.f;
     }
     const float* prow = a.p + (long long)h * D;
+    // one group of copies is committed for every stage, empty past the end, so the count to wait for is fixed
     auto fetch = [&](int base, int buf) {
-        const int cnt = min(TT, t1 - base);
+        const int cnt = max(0, min(TT, t1 - base));
         const int vcols = min(COLS, E - j0);                   // (<= 0: this block has the column behind the values only)
         if (VEC) {
             const int n4 = D >> 2;
@@ -285,27 +306,24 @@ lin_scan_kernel(ScanParams a, LinShape s) {
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    const bool busy = j0 + warp * (32 / SCAN_LANES) * C < EW;  // a warp whose columns lie past the end only helps fetching
-    const bool sums_decay = PASS == SCAN_SUM && blockIdx.x == 0 && warp == 0;
-    uint64_t total[NC][2];
-    float total_h = 1.f;
+    const bool busy = j0 + warp * (32 / LANES) * C < EW;  // a warp whose columns lie past the end only helps fetching
+    const bool sums_decay = PASS == SCAN_SUM && blockIdx.x == 0;       // the chunk's total decay: of channels tid and tid + 128, or of the head
+    float total[2] = {1.f, 1.f};
+    // behind the exchange a lane holds the sum of one of the C columns: the bits of its number from the top
+    constexpr int SPARE = LANES / C;                           // lanes that end with the same column
+    int my_x = 0;
 #pragma unroll
-    for (int c = 0; c < NC; ++c) total[c][0] = total[c][1] = pair_of(1.f, 1.f);
-    // after the exchange below a lane holds the sum of one of the C columns
-    const int my_x = C == 4 ? ((l >> 2) & 1) * 2 + ((l >> 1) & 1) : (l >> 2) & 1;
-    const bool stores = C == 4 ? (l & 1) == 0 : (l & 3) == 0;
+    for (int n = C / 2, mask = LANES / 2; n >= 1; n >>= 1, mask >>= 1) my_x += (l & mask) ? n : 0;
+    const bool stores = l % SPARE == 0;
 
-    fetch(t0, 0);
+#pragma unroll
+    for (int i = 0; i < ST - 1; ++i) fetch(t0 + i * TT, i);
     int buf = 0;
-    for (int base = t0; base < t1; base += TT, buf ^= 1) {
+    for (int base = t0; base < t1; base += TT, buf = buf + 1 == ST ? 0 : buf + 1) {
         const int cnt = min(TT, t1 - base);
-        if (base + TT < t1) {
-            fetch(base + TT, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
+        asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+        __syncthreads();                                       // this stage is there, and nobody reads the one before it any more
+        fetch(base + (ST - 1) * TT, buf == 0 ? ST - 1 : buf - 1);
         auto token = [&](int tt) {
             const float* vt = sv + (buf * TT + tt) * COLS + col;
             float v[C];
@@ -317,7 +335,6 @@ lin_scan_kernel(ScanParams a, LinShape s) {
                 keep2 = pair_of(g.x, g.x);
 #pragma unroll
                 for (int x = 0; x < C; ++x) v[x] *= g.y;
-                if (sums_decay) total_h *= g.x;
             }
             uint64_t v2[C], o2[C];
 #pragma unroll
@@ -327,10 +344,10 @@ lin_scan_kernel(ScanParams a, LinShape s) {
             const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(sa + (buf * TT + tt) * DP);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                const ulonglong2 kk = k4[c * SCAN_LANES + l];
+                const ulonglong2 kk = k4[c * LANES + l];
                 ulonglong2 qq, aa;
-                if (PASS != SCAN_SUM) qq = q4[c * SCAN_LANES + l];
-                if (!HEAD) aa = a4[c * SCAN_LANES + l];
+                if (PASS != SCAN_SUM) qq = q4[c * LANES + l];
+                if (!HEAD) aa = a4[c * LANES + l];
                 const uint64_t k2[2] = {kk.x, kk.y};
                 const uint64_t a2[2] = {HEAD ? keep2 : aa.x, HEAD ? keep2 : aa.y};
 #pragma unroll
@@ -340,31 +357,25 @@ lin_scan_kernel(ScanParams a, LinShape s) {
                         st[c][u][x] = fma_pair(a2[u], st[c][u][x], mul_pair(k2[u], v2[x]));
                         if (PASS != SCAN_SUM) o2[x] = fma_pair(st[c][u][x], u ? qq.y : qq.x, o2[x]);
                     }
-                    if (!HEAD && sums_decay) total[c][u] = mul_pair(total[c][u], a2[u]);
                 }
             }
             if (PASS != SCAN_SUM) {
                 float o[C];
 #pragma unroll
                 for (int x = 0; x < C; ++x) { float lo, hi; halves_of(o2[x], lo, hi); o[x] = lo + hi; }
-                // the eight lanes' shares: each exchange halves the columns a lane is left with
-                float r;
-                if (C == 4) {
-                    const bool up = l & 4;
-                    const float k0 = up ? o[2] : o[0], k1 = up ? o[3] : o[1], g0 = up ? o[0] : o[2], g1 = up ? o[1] : o[3];
-                    const float e0 = k0 + __shfl_xor_sync(0xffffffffu, g0, 4), e1 = k1 + __shfl_xor_sync(0xffffffffu, g1, 4);
-                    const bool odd = l & 2;
-                    r = (odd ? e1 : e0) + __shfl_xor_sync(0xffffffffu, odd ? e0 : e1, 2);
-                    r += __shfl_xor_sync(0xffffffffu, r, 1);
-                } else {
-                    const bool up = l & 4;
-                    r = (up ? o[1] : o[0]) + __shfl_xor_sync(0xffffffffu, up ? o[0] : o[1], 4);
-                    r += __shfl_xor_sync(0xffffffffu, r, 2);
-                    r += __shfl_xor_sync(0xffffffffu, r, 1);
-                }
+                const float r = lane_sums<LANES, C>(o, l);
                 if (stores && j + my_x < EW) a.out[((long long)(base + tt) * H + h) * EW + j + my_x] = r;
             }
         };
+        if (PASS == SCAN_SUM && sums_decay) {
+            for (int tt = 0; tt < cnt; ++tt) {
+                if (HEAD) total[0] *= sg[(buf * TT + tt) * 4];
+                else {
+                    if (tid < DP) total[0] *= sa[(buf * TT + tt) * DP + tid];
+                    if (DP > 128 && tid + 128 < DP) total[1] *= sa[(buf * TT + tt) * DP + tid + 128];
+                }
+            }
+        }
         if (busy) {
             if (cnt == TT) {
 #pragma unroll
@@ -373,14 +384,22 @@ lin_scan_kernel(ScanParams a, LinShape s) {
                 for (int tt = 0; tt < cnt; ++tt) token(tt);
             }
         }
-        __syncthreads();                                       // this buffer is asked for again in the next turn
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (PASS == SCAN_SUM && sums_decay) {
+        float* P = a.decay + (((long long)ck * a.n_seqs + b) * H + h) * (HEAD ? 1 : D);
+        if (HEAD) { if (tid == 0) *P = total[0]; }
+        else {
+            if (tid < D) P[tid] = total[0];
+            if (tid + 128 < D) P[tid + 128] = total[1];
+        }
     }
     if (!busy || (PASS == SCAN_OUT && t1 != s1)) return;
 #pragma unroll
     for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
-            const int d = (c * SCAN_LANES + l) * 4 + 2 * u;
+            const int d = (c * LANES + l) * 4 + 2 * u;
 #pragma unroll
             for (int x = 0; x < C; ++x) {
                 float v0, v1;
@@ -389,15 +408,7 @@ lin_scan_kernel(ScanParams a, LinShape s) {
                 if (d < D) *(PASS == SCAN_SUM ? Wh + (long long)d * EW + j + x : place(d, j + x)) = v0;
                 if (d + 1 < D) *(PASS == SCAN_SUM ? Wh + (long long)(d + 1) * EW + j + x : place(d + 1, j + x)) = v1;
             }
-            if (!HEAD && sums_decay && tid < SCAN_LANES) {
-                float v0, v1;
-                halves_of(total[c][u], v0, v1);
-                float* P = a.decay + (((long long)ck * a.n_seqs + b) * H + h) * D;
-                if (d < D) P[d] = v0;
-                if (d + 1 < D) P[d + 1] = v1;
-            }
         }
-    if (HEAD && sums_decay && tid == 0) a.decay[((long long)ck * a.n_seqs + b) * H + h] = total_h;
 }
 
 // Chunk contributions -> the state before every chunk, in place: one thread a (sequence, head, channel, column).
@@ -456,32 +467,36 @@ lin_finish_kernel(const float* __restrict__ o, int EW, const float* __restrict__
     float factor = q_scale;
     if (s.head_form) factor = q_scale / (fmaxf(fabsf(q_scale * orow[E]), floor_[wid]) + 1e-6f);
     constexpr int KEEP = 8;                                    // values a lane keeps between the passes
-    float v[KEEP];
+    float v[KEEP], zk[KEEP];
     float ss = 0.f;
 #pragma unroll
-    for (int u = 0; u < KEEP; ++u) {
+    for (int u = 0; u < KEEP; ++u) {                           // (the gate's sums are asked for together with the values)
         const int e = lane + 32 * u;
-        v[u] = e < E ? orow[e] * factor : 0.f;
+        v[u] = e < E ? orow[e] : 0.f;
+        zk[u] = e < E ? p[t * s.ldp + s.g_off + h * E + e] : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < KEEP; ++u) {
+        v[u] *= factor;
         ss = fmaf(v[u], v[u], ss);
     }
     for (int e = lane + 32 * KEEP; e < E; e += 32) { const float x = orow[e] * factor; ss = fmaf(x, x, ss); }
     const float inv = inv_rms(warp_sum(ss), (float)E, eps) * out_scale;
     if (w_heads) w += (long long)h * E;
-    auto put = [&](int e, float x) {
-        const float z = lin_at(p, s, t, s.g_off + h * E + e);
+    auto put = [&](int e, float x, float z) {
         const float g = sigmoid_(z);
         out[wid * E + e] = from_f32<TO>(x * inv * w[e] * (silu_gate ? z * g : g));
     };
 #pragma unroll
     for (int u = 0; u < KEEP; ++u) {
         const int e = lane + 32 * u;
-        if (e < E) put(e, v[u]);
+        if (e < E) put(e, v[u], zk[u]);
     }
-    for (int e = lane + 32 * KEEP; e < E; e += 32) put(e, orow[e] * factor);
+    for (int e = lane + 32 * KEEP; e < E; e += 32) put(e, orow[e] * factor, p[t * s.ldp + s.g_off + h * E + e]);
 }
 
 // ---------------------------------------------------------------------------------------
-// one token a sequence: everything between the input product and the output product in one kernel, a block a (head, sequence)
+// one token a sequence: everything between the input product and the output product in one kernel
 // ---------------------------------------------------------------------------------------
 struct StepParams {
     const float* p;
@@ -496,31 +511,50 @@ struct StepParams {
 
 constexpr int STEP_THREADS = 256;
 constexpr int STEP_AHEAD = 8;                 // 16-byte pieces of the state a thread asks for before the kernel ahead has ended
+constexpr int STEP_PARTS = 8;                 // the most blocks that share a head (a cluster)
 
+__device__ __forceinline__ void cluster_meet() {
+    asm volatile("barrier.cluster.arrive.release;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire;" ::: "memory");
+}
+// the float at ``p`` (shared memory) of the cluster's block ``rank``
+__device__ __forceinline__ float cluster_read(const float* p, int rank) {
+    uint32_t a;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
+    return v;
+}
+
+// Grid (parts, heads, sequences), clusters of ``parts`` blocks: a block takes ``cols`` columns of its head's S.  The blocks of a
+// cluster meet once, for the sum of squares over the whole head; what they all need (q, k, gates, n.q) each works out itself, and
+// the first one writes n and m once the others have read them.
 template <typename TO, bool VEC>
-__global__ void __launch_bounds__(STEP_THREADS)
-lin_step_kernel(StepParams a, LinShape s) {
+__global__ void __launch_bounds__(STEP_THREADS, 2)
+lin_step_kernel(StepParams a, LinShape s, int cols) {
     constexpr int W = VEC ? 4 : 1;
     extern __shared__ __align__(16) float sm[];
-    const int D = s.D, E = s.E, H = s.H;
-    const int EP = (E + 3) / 4 * 4;
+    const int D = s.D, H = s.H, parts = gridDim.x, part = blockIdx.x;
+    const int c0 = part * cols, E = min(cols, s.E - c0);       // this block's columns
+    const int EP = (cols + 3) / 4 * 4, ER = (E + 3) / 4 * 4;
     float* sq = sm;                            // [D]
     float* sk = sq + D;                        // [D]
     float* sa = sk + D;                        // [D] decays (channel form)
     float* sv = sa + D + (4 - 3 * D % 4) % 4;  // [EP]
     float* sz = sv + EP;                       // [EP] the output gate's sums
-    float* red = sz + EP;                      // [groups][EP]
-    __shared__ float rs[40], low[MAX_RANK];
+    float* red = sz + EP;                      // [groups][ER]: at most max(4 * STEP_THREADS, EP) numbers
+    __shared__ float rs[40], low[MAX_RANK], shared_ss;
     pdl_trigger();
-    const int tid = threadIdx.x, h = blockIdx.x, b = blockIdx.y;
+    const int tid = threadIdx.x, h = blockIdx.y, b = blockIdx.z;
     const long long slot = a.seq_slot[b];
     const long long t = a.seq_start[b];
-    float* Sh = a.S + (slot * H + h) * D * E;
-    const int ne = E / W;                      // pieces of a row of S
-    const int per = ne < STEP_THREADS ? ne : STEP_THREADS;     // threads on one row
+    float* Sh = a.S + (slot * H + h) * D * s.E + c0;
+    float* nh = s.head_form ? a.n + (slot * H + h) * D : nullptr;
+    const int ne = E / W;                      // pieces of a row of this block's columns
+    const int per = max(1, min(ne, STEP_THREADS));             // threads on one row
     const int groups = STEP_THREADS / per;     // rows side by side
     const int grp = tid / per, e0 = tid % per;
-    const bool works = grp < groups;
+    const bool works = grp < groups && ne > 0;
     // the state was left by an earlier step: its first pieces are asked for while the kernel ahead still runs
     alignas(16) float ahead[STEP_AHEAD][W];
     if (works) {
@@ -528,55 +562,73 @@ lin_step_kernel(StepParams a, LinShape s) {
         for (int u = 0; u < STEP_AHEAD; ++u) {
             const int d = grp + u * groups;
             if (d < D) {
-                if (VEC) *reinterpret_cast<float4*>(ahead[u]) = *reinterpret_cast<const float4*>(Sh + (long long)d * E + e0 * W);
-                else ahead[u][0] = Sh[(long long)d * E + e0];
+                if (VEC) *reinterpret_cast<float4*>(ahead[u]) = *reinterpret_cast<const float4*>(Sh + (long long)d * s.E + e0 * W);
+                else ahead[u][0] = Sh[(long long)d * s.E + e0];
             }
         }
     }
+    const float n_old = (s.head_form && tid < D) ? nh[tid] : 0.f;              // (D <= 256: a channel a thread)
+    const float m_old = s.head_form ? a.m[slot * H + h] : 0.f;
+    static_assert(STEP_THREADS >= 256, "a key channel a thread");
     pdl_wait();
-    for (int i = tid; i < 2 * D; i += STEP_THREADS) {
-        const int d = i < D ? i : i - D;
-        sq[i] = lin_at(a.p, s, t, (i < D ? s.q_off : s.k_off) + h * D + d);          // (q and k lie one behind the other)
+    // everything this block needs of the projection row, several numbers a thread asked for before the first is put away:
+    // q, k, this block's columns of v and of the output gate, and the gates' sums or the low-rank columns
+    const int n_low = s.head_form ? 2 : s.rank, total = 2 * D + 2 * E + n_low;
+    auto column = [&](int i, float*& dst) -> int {
+        if (i < D) { dst = sq + i; return s.q_off + h * D + i; }
+        i -= D;
+        if (i < D) { dst = sk + i; return s.k_off + h * D + i; }
+        i -= D;
+        if (i < E) { dst = sv + i; return s.v_off + h * s.E + c0 + i; }
+        i -= E;
+        if (i < E) { dst = sz + i; return s.g_off + h * s.E + c0 + i; }
+        i -= E;
+        dst = low + i;
+        return s.head_form ? (i == 0 ? s.x_off : s.y_off) + h : s.x_off + i;
+    };
+    for (int i0 = tid; i0 < total; i0 += 4 * STEP_THREADS) {
+        float v[4];
+        float* dst[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int i = i0 + u * STEP_THREADS;
+            dst[u] = nullptr;
+            if (i < total) v[u] = lin_at(a.p, s, t, column(i, dst[u]));
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+            if (dst[u]) *dst[u] = v[u];
     }
-    for (int i = tid; i < 2 * E; i += STEP_THREADS) {
-        const int e = i < E ? i : i - E;
-        (i < E ? sv : sz)[e] = lin_at(a.p, s, t, (i < E ? s.v_off : s.g_off) + h * E + e);
-    }
-    float keep = 1.f, put = 1.f, floor_ = 0.f, m_new = 0.f;
+    __syncthreads();
+    float keep = 1.f, put = 1.f, floor_ = 0.f;
     if (s.head_form) {
         if (tid == 0) {
             float li, lf;
-            log_gates(a.p, s, t, h, a.bi, a.bf, a.cap, li, lf);
-            const float m = a.m[slot * H + h];
-            m_new = fmaxf(lf + m, li);
-            rs[34] = expf(lf + m - m_new);
+            log_gates(low[0] + a.bi[h], low[1] + a.bf[h], a.cap, li, lf);
+            const float m_new = fmaxf(lf + m_old, li);
+            rs[34] = expf(lf + m_old - m_new);
             rs[35] = expf(li - m_new);
             rs[36] = expf(-m_new);
-            a.m[slot * H + h] = m_new;
+            rs[37] = m_new;
         }
-    } else {
-        for (int r = tid; r < s.rank; r += STEP_THREADS) low[r] = lin_at(a.p, s, t, s.x_off + r);
     }
-    __syncthreads();
-    if (s.head_form) {
-        keep = rs[34]; put = rs[35]; floor_ = rs[36];
-    } else {
+    if (!s.head_form) {
         for (int d = tid; d < D; d += STEP_THREADS) {
             const int c = h * D + d;
             float z = 0.f;
+#pragma unroll 8
             for (int r = 0; r < s.rank; ++r) z = fmaf(a.up[(long long)r * H * D + c], low[r], z);
             sa[d] = expf(log_sigmoid_(z + a.bias[c]) * a.inv_tau);
         }
-        __syncthreads();
     }
+    __syncthreads();
+    if (s.head_form) { keep = rs[34]; put = rs[35]; floor_ = rs[36]; }
     // the vector n and its product with q
-    float nq = 0.f;
+    float nq = 0.f, n_new = 0.f;
     if (s.head_form) {
-        float* nh = a.n + (slot * H + h) * D;
-        for (int d = tid; d < D; d += STEP_THREADS) {
-            const float x = fmaf(keep, nh[d], put * sk[d]);
-            nh[d] = x;
-            nq = fmaf(x, sq[d], nq);
+        if (tid < D) {
+            n_new = fmaf(keep, n_old, put * sk[tid]);
+            nq = n_new * sq[tid];
         }
         nq = block_sum(nq, rs);
     }
@@ -594,8 +646,8 @@ lin_step_kernel(StepParams a, LinShape s) {
                     x[y] = fmaf(dk, x[y], k * v[y]);
                     acc[y] = fmaf(x[y], q, acc[y]);
                 }
-                if (VEC) *reinterpret_cast<float4*>(Sh + (long long)d * E + ee * W) = *reinterpret_cast<float4*>(x);
-                else Sh[(long long)d * E + ee] = x[0];
+                if (VEC) *reinterpret_cast<float4*>(Sh + (long long)d * s.E + ee * W) = *reinterpret_cast<float4*>(x);
+                else Sh[(long long)d * s.E + ee] = x[0];
             };
             int d = grp;
             if (eb == 0) {
@@ -605,22 +657,22 @@ lin_step_kernel(StepParams a, LinShape s) {
                     d += groups;
                 }
             }
-            for (; d < D; d += 4 * groups) {
-                alignas(16) float x[4][W];
+            for (; d < D; d += 8 * groups) {
+                alignas(16) float x[8][W];
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
+                for (int u = 0; u < 8; ++u) {
                     const int dd = d + u * groups;
                     if (dd < D) {
-                        if (VEC) *reinterpret_cast<float4*>(x[u]) = *reinterpret_cast<const float4*>(Sh + (long long)dd * E + ee * W);
-                        else x[u][0] = Sh[(long long)dd * E + ee];
+                        if (VEC) *reinterpret_cast<float4*>(x[u]) = *reinterpret_cast<const float4*>(Sh + (long long)dd * s.E + ee * W);
+                        else x[u][0] = Sh[(long long)dd * s.E + ee];
                     }
                 }
 #pragma unroll
-                for (int u = 0; u < 4; ++u)
+                for (int u = 0; u < 8; ++u)
                     if (d + u * groups < D) row(d + u * groups, x[u]);
             }
 #pragma unroll
-            for (int y = 0; y < W; ++y) red[(long long)grp * EP + ee * W + y] = acc[y];
+            for (int y = 0; y < W; ++y) red[grp * ER + ee * W + y] = acc[y];
         }
     }
     __syncthreads();
@@ -629,18 +681,30 @@ lin_step_kernel(StepParams a, LinShape s) {
     float ss = 0.f;
     for (int e = tid; e < E; e += STEP_THREADS) {
         float o = 0.f;
-        for (int g = 0; g < groups; ++g) o += red[(long long)g * EP + e];
+        for (int g = 0; g < groups; ++g) o += red[g * ER + e];
         o *= factor;
         sv[e] = o;                              // (v is used up)
         ss = fmaf(o, o, ss);
     }
-    const float inv = inv_rms(block_sum(ss, rs), (float)E, a.eps) * a.out_scale;
-    const float* w = a.w + (a.w_heads ? (long long)h * E : 0);
-    TO* out = (TO*)a.out + (t * H + h) * E;
+    ss = block_sum(ss, rs);
+    if (parts > 1) {
+        if (tid == 0) shared_ss = ss;
+        cluster_meet();                         // every block's share is there, and every block has read n and m
+        ss = 0.f;
+        for (int r = 0; r < parts; ++r) ss += cluster_read(&shared_ss, r);
+    }
+    if (s.head_form && part == 0) {
+        if (tid < D) nh[tid] = n_new;
+        if (tid == 0) a.m[slot * H + h] = rs[37];
+    }
+    const float inv = inv_rms(ss, (float)s.E, a.eps) * a.out_scale;
+    const float* w = a.w + (a.w_heads ? (long long)h * s.E : 0) + c0;
+    TO* out = (TO*)a.out + (t * H + h) * s.E + c0;
     for (int e = tid; e < E; e += STEP_THREADS) {
         const float z = sz[e], g = sigmoid_(z);
         out[e] = from_f32<TO>(sv[e] * inv * w[e] * (a.silu_gate ? z * g : g));
     }
+    if (parts > 1) cluster_meet();              // no block leaves while another may still read its share
 }
 
 // ---------------------------------------------------------------------------------------
@@ -676,12 +740,12 @@ UB_API int ub_lin_gates(const float* p, long long ldp, int n_parts, long long pa
                                     seq_start, seq_slot, keep, put, floor_);
 }
 
-template <int R, int C, bool HEAD, bool VEC, int PASS>
+template <int LANES, int R, int C, bool HEAD, bool VEC, int PASS>
 static cudaError_t launch_scan(const ScanParams& a, const LinShape& s, cudaStream_t st) {
-    using L = ScanLayout<R, C, HEAD>;
+    using L = ScanLayout<LANES, R, C, HEAD>;
     static bool attr_done = false;
     if (!attr_done && L::BYTES > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(lin_scan_kernel<R, C, HEAD, VEC, PASS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES);
+        cudaError_t e = cudaFuncSetAttribute(lin_scan_kernel<LANES, R, C, HEAD, VEC, PASS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L::BYTES);
         if (e != cudaSuccess) return e;
         attr_done = true;
     }
@@ -689,18 +753,18 @@ static cudaError_t launch_scan(const ScanParams& a, const LinShape& s, cudaStrea
     const dim3 grid((a.EW + L::COLS - 1) / L::COLS, s.H, a.n_seqs * chunks);
     // an ordinary launch: as a programmatic dependent the blocks, each busy for the whole kernel, would be placed several to an
     // SM on the SMs that the kernel before leaves first
-    return ub_launch_ordered(false, lin_scan_kernel<R, C, HEAD, VEC, PASS>, grid, dim3(128), L::BYTES, st, a, s);
+    return ub_launch_ordered(false, lin_scan_kernel<LANES, R, C, HEAD, VEC, PASS>, grid, dim3(128), L::BYTES, st, a, s);
 }
 
-template <int R, int C, bool HEAD, bool VEC>
+template <int LANES, int R, int C, bool HEAD, bool VEC>
 static cudaError_t scan_all(const ScanParams& a, const LinShape& s, cudaStream_t st) {
-    if (a.n_chunks <= 1) return launch_scan<R, C, HEAD, VEC, SCAN_WHOLE>(a, s, st);
-    cudaError_t e = launch_scan<R, C, HEAD, VEC, SCAN_SUM>(a, s, st);
+    if (a.n_chunks <= 1) return launch_scan<LANES, R, C, HEAD, VEC, SCAN_WHOLE>(a, s, st);
+    cudaError_t e = launch_scan<LANES, R, C, HEAD, VEC, SCAN_SUM>(a, s, st);
     if (e != cudaSuccess) return e;
     const long long n = (long long)a.n_seqs * s.H * s.D * a.EW;
     e = ub_launch_dependent(lin_carry_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, a, s.H, s.D, s.E, s.head_form);
     if (e != cudaSuccess) return e;
-    return launch_scan<R, C, HEAD, VEC, SCAN_OUT>(a, s, st);
+    return launch_scan<LANES, R, C, HEAD, VEC, SCAN_OUT>(a, s, st);
 }
 
 // The projection whole (one part).  ``n_chunks`` chunks of ``chunk`` tokens cover the longest sequence (1: no chunks; work and
@@ -718,21 +782,17 @@ UB_API int ub_lin_scan(const float* p, long long ldp, const int* shape, const fl
                  n_seqs, n_chunks, chunk};
     const bool vec = s.D % 4 == 0 && s.E % 4 == 0 && ldp % 4 == 0 && (s.q_off | s.k_off | s.v_off) % 4 == 0 &&
         (((uintptr_t)p | (uintptr_t)(s.head_form ? nullptr : dec)) & 15) == 0;
-    const int per_lane = (s.D + SCAN_LANES - 1) / SCAN_LANES;
     cudaError_t e;
-#define GO2(RR, CC, HH) e = vec ? scan_all<RR, CC, HH, true>(a, s, st) : scan_all<RR, CC, HH, false>(a, s, st)
-#define GO(RR, CC) do { if (s.head_form) GO2(RR, CC, true); else GO2(RR, CC, false); } while (0)
-    if (per_lane <= 4) GO(4, 4);
-    else if (per_lane <= 8) GO(8, 4);
-    else if (per_lane <= 16) GO(16, 4);
-    else GO(32, 2);
+#define GO2(LL, RR, CC, HH) e = vec ? scan_all<LL, RR, CC, HH, true>(a, s, st) : scan_all<LL, RR, CC, HH, false>(a, s, st)
+#define GO(LL, RR, CC) do { if (s.head_form) GO2(LL, RR, CC, true); else GO2(LL, RR, CC, false); } while (0)
+    if (s.D <= 32) GO(8, 4, 8);                                // (blocks of 128 columns, 128, 64 and 32: lin_chunks counts them)
+    else if (s.D <= 64) GO(8, 8, 8);
+    else if (s.D <= 128) GO(8, 16, 4);
+    else GO(32, 8, 8);
 #undef GO
 #undef GO2
     return (int)e;
 }
-
-// Columns of S a block of the scan takes.
-UB_API int ub_lin_scan_cols(int D) { return (D + SCAN_LANES - 1) / SCAN_LANES <= 16 ? 64 : 32; }
 
 UB_API int ub_lin_finish(const float* o, const float* p, long long ldp, const int* shape, const float* floor_, const float* w,
                          int w_heads, int silu_gate, void* out, int out_dtype, int n_tokens, float q_scale, float eps,
@@ -754,7 +814,7 @@ UB_API int ub_lin_finish(const float* o, const float* p, long long ldp, const in
 UB_API int ub_lin_step(const float* p, long long ldp, int n_parts, long long part_stride, const int* shape, const float* up,
                        const float* bias, float tau, const float* bi, const float* bf, float cap, float* S, float* n, float* m,
                        const int* seq_start, const int* seq_slot, const float* w, int w_heads, int silu_gate, void* out,
-                       int out_dtype, int n_seqs, float q_scale, float eps, float out_scale, cudaStream_t st) {
+                       int out_dtype, int n_seqs, float q_scale, float eps, float out_scale, int sm_count, cudaStream_t st) {
     if (n_seqs <= 0) return 0;
     LinShape s;
     if (int rc = read_shape(shape, ldp, n_parts, part_stride, s)) return rc;
@@ -763,14 +823,31 @@ UB_API int ub_lin_step(const float* p, long long ldp, int n_parts, long long par
     StepParams a{p, up, bias, s.head_form ? 0.f : 1.0f / tau, bi, bf, cap, S, n, m, seq_start, seq_slot, w, w_heads, silu_gate, out,
                  q_scale, eps, out_scale};
     const bool vec = s.E % 4 == 0 && ((uintptr_t)S & 15) == 0;
-    const int ne = vec ? s.E / 4 : s.E, per = ne < STEP_THREADS ? ne : STEP_THREADS, EP = (s.E + 3) / 4 * 4;
-    const size_t smem = ((size_t)3 * s.D + 4 + (2 + STEP_THREADS / per) * (size_t)EP) * sizeof(float);
-    const dim3 grid(s.H, n_seqs);
+    // blocks that share a head: as many as the SMs hold at once, two each (at least 16 columns a block, and none without any)
+    int parts = 1;
+    const int width = vec ? 4 : 1;
+    auto cols_of = [&](int n) { return ((s.E + n - 1) / n + width - 1) / width * width; };
+    while (parts < STEP_PARTS && cols_of(2 * parts) >= 16 && (2 * parts - 1) * cols_of(2 * parts) < s.E &&
+           2LL * parts * s.H * n_seqs <= 2LL * (sm_count > 0 ? sm_count : 148)) parts *= 2;
+    const int cols = cols_of(parts);
+    const int EP = (cols + 3) / 4 * 4;
+    const size_t smem = ((size_t)3 * s.D + 4 + 2 * (size_t)EP + (EP > 4 * STEP_THREADS ? EP : 4 * STEP_THREADS)) * sizeof(float);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(parts, s.H, n_seqs);
+    cfg.blockDim = dim3(STEP_THREADS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = parts;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    static const int plain = [] { const char* v = getenv("ULTIMA_PDL"); return v && v[0] == '0'; }();   // for measurements
+    cfg.attrs = attr;
+    cfg.numAttrs = plain ? 1 : 2;
     cudaError_t e;
-#define GO(TO, VV) do { static bool done = false; \
-        if (!done && smem > 48 * 1024) { e = cudaFuncSetAttribute(lin_step_kernel<TO, VV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
-            if (e != cudaSuccess) return (int)e; done = true; } \
-        e = ub_launch_dependent(lin_step_kernel<TO, VV>, grid, dim3(STEP_THREADS), smem, st, a, s); } while (0)
+#define GO(TO, VV) e = cudaLaunchKernelEx(&cfg, lin_step_kernel<TO, VV>, a, s, cols)
     if (out_dtype == UB_F32) { if (vec) GO(float, true); else GO(float, false); }
     else if (out_dtype == UB_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
     else return UB_ERR_UNSUPPORTED;

@@ -40,8 +40,15 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
     const float* bias = (mode & 16) ? corr : nullptr;
     if (mode & 16) corr = nullptr;
     for (int i = lane; i < n_out; i += 32) {              // the logits may come as K slices: summed in the slices' order
-        float v = zr[i];
-        for (int s = 1; s < n_parts; ++s) v += zr[s * part_stride + i];
+        float v = 0.f;
+        for (int s0 = 0; s0 < n_parts; s0 += 8) {         // eight slices asked for at a time
+            float part[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u) part[u] = s0 + u < n_parts ? zr[(s0 + u) * part_stride + i] : 0.f;
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                if (s0 + u < n_parts) v = s0 + u == 0 ? part[u] : v + part[u];
+        }
         if (bias) v += bias[i];
         sc[i] = v;
         m = fmaxf(m, v);
@@ -178,16 +185,21 @@ route_small_kernel(const float* __restrict__ z, long long ldz, int n_parts, long
         __syncwarp();
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
+    if (warp == 0) {                                            // running sums over the experts, 32 at a time
         int row = 0, tl = 0;
-        for (int e = 0; e < n_experts; ++e) {
-            seg[e] = row;
-            first_tile[e] = tl;
-            row += cnt[e];
-            tl += (cnt[e] + tile - 1) / tile;
+        for (int e0 = 0; e0 < n_experts; e0 += 32) {
+            const int e = e0 + lane, n = e < n_experts ? cnt[e] : 0, k = (n + tile - 1) / tile;
+            int rs = n, ts = k;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int pr = __shfl_up_sync(0xffffffffu, rs, o), pt = __shfl_up_sync(0xffffffffu, ts, o);
+                if (lane >= o) { rs += pr; ts += pt; }
+            }
+            if (e < n_experts) { seg[e] = row + rs - n; first_tile[e] = tl + ts - k; }
+            row += __shfl_sync(0xffffffffu, rs, 31);
+            tl += __shfl_sync(0xffffffffu, ts, 31);
         }
-        first_tile[n_experts] = tl;
-        *n_tiles = tl;
+        if (lane == 0) { first_tile[n_experts] = tl; *n_tiles = tl; }
     }
     __syncthreads();
     for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {

@@ -153,9 +153,8 @@ def _declare(lib, source: str) -> None:
         "linear.cu": {"ub_lin_decay": [P, L, I, L, P, P, P, P, I, F, P],
                       "ub_lin_gates": [P, L, I, L, P, P, P, F, P, P, P, I, P, P, P, P],
                       "ub_lin_scan": [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, P],
-                      "ub_lin_scan_cols": [I],
                       "ub_lin_finish": [P, P, L, P, P, P, I, I, P, I, I, F, F, F, P],
-                      "ub_lin_step": [P, L, I, L, P, P, P, F, P, P, F, P, P, P, P, P, P, I, I, P, I, I, F, F, F, P]},
+                      "ub_lin_step": [P, L, I, L, P, P, P, F, P, P, F, P, P, P, P, P, P, I, I, P, I, I, F, F, F, I, P]},
         "sampling.cu": {"ub_sample": [P, L, P, I, I, P, P, P, P, P, U, P, P, I, P], "ub_sample_params_size": []},
     }.get(source, {})
     for name, args in sigs.items():
@@ -877,16 +876,19 @@ def lin_gates(p, form, b_in, b_forget, cap, m, batch, keep, put, floor):
 
 
 LIN_CHUNK = 64              # the fewest tokens a chunk of the scan has
-LIN_BLOCKS = 6              # blocks an SM the scan is cut into chunks for
+LIN_CTAS = 3                # blocks of the scan that an SM holds
 
 
 def lin_chunks(form, n_seqs: int, max_new: int, n_sms: int | None = None):
-    """(chunks, tokens a chunk) of a step whose longest sequence brings ``max_new`` tokens: as many chunks as fill the GPU, and
-    none at all where cutting would not pay for doing the state's update twice."""
-    cols = 64 if form.D <= 128 else 32
-    blocks = n_seqs * form.H * -(-form.E // cols)
-    want = -(-LIN_BLOCKS * (n_sms or sm_count()) // blocks)
-    n = min(want, max_new // LIN_CHUNK, 65535 // max(1, n_seqs))
+    """(chunks, tokens a chunk) of a step whose longest sequence brings ``max_new`` tokens.  Cutting costs the state's update twice,
+    so it is for steps that would leave SMs empty; there a few whole waves of blocks, in at least eight chunks."""
+    cols = 128 if form.D <= 64 else 64 if form.D <= 128 else 32
+    blocks = n_seqs * form.H * -(-(form.E + (1 if form.head_form else 0)) // cols)
+    sms = n_sms or sm_count()
+    if blocks >= sms:
+        return 1, max(1, max_new)
+    waves = -(-8 * blocks // (LIN_CTAS * sms))
+    n = min(waves * LIN_CTAS * sms // blocks, max_new // LIN_CHUNK, 65535 // max(1, n_seqs))
     if n < 4:
         return 1, max(1, max_new)
     chunk = -(-max_new // n)
@@ -955,7 +957,7 @@ def lin_step(p, form, state, batch, weight, out, q_scale, eps, out_scale=1.0, si
     _check(_lib("linear.cu").ub_lin_step(_ptr(p), ldp, n_parts, part_stride, form.ints, _ptr(up), _ptr(bias), float(tau), _ptr(bi),
                                          _ptr(bf), float(cap), _ptr(S), _ptr(n), _ptr(m), _ptr(batch.seq_start), _ptr(batch.seq_slot),
                                          _ptr(weight), 1 if weight.numel() == H * E and H > 1 else 0, 1 if silu_gate else 0, _ptr(out),
-                                         _code(out), T, float(q_scale), float(eps), float(out_scale), _stream()), "lin_step")
+                                         _code(out), T, float(q_scale), float(eps), float(out_scale), sm_count(), _stream()), "lin_step")
 
 
 # ---------------------------------------------------------------------------------------
