@@ -368,6 +368,39 @@ def test_one_token_a_sequence_in_one_kernel(H, D, E, dtype):
 # ---------------------------------------------------------------------------------------
 # attention with values of another size
 # ---------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("nh,nkv,hd,hdv", [(4, 2, 32, 48), (3, 1, 20, 28), (2, 2, 64, 128), (16, 4, 64, 128), (32, 8, 128, 128), (3, 3, 10, 14), (5, 5, 9, 4)])
+def test_placement_with_a_norm_over_all_heads(nh, nkv, hd, hdv, dtype):
+    """Sizes in fours (rows in registers, of every length the kernel is built for) and others; the projection whole, in slices, and
+    as columns of wider rows; two sequences on a ring that wraps."""
+    import plain_demazen as P
+    ops = _ops()
+    qn, kn, vn, T, eps = nh * hd, nkv * hd, nkv * hdv, 70, 1e-3
+    g = torch.Generator().manual_seed(qn)
+    qw, kw = 1 + 0.2 * torch.randn(qn, generator=g), 1 + 0.2 * torch.randn(kn, generator=g)
+    pos = torch.cat([torch.arange(40) + 100, torch.arange(30)]).to(torch.int32)
+    seq = torch.tensor([0] * 40 + [1] * 30, dtype=torch.int32)
+    table = torch.tensor([[4, 1], [0, 3]], dtype=torch.int32)
+    for parts, pad in ((1, 0), (3, 0), (1, 8), (2, 4)):
+        xs = torch.randn(parts, T, qn + kn + vn + pad, generator=g)
+        x = xs.sum(0).double()
+        dev = xs.to(DEV)[..., :qn + kn + vn]
+        q = torch.full((T, qn), float("nan"), dtype=dtype, device=DEV)
+        kc = torch.full((5, nkv, 64, hd), 9.0, dtype=dtype, device=DEV)
+        vc = torch.full((5, nkv, 64, hdv), 9.0, dtype=dtype, device=DEV)
+        ops.qkv_place_rows(dev if parts > 1 else dev[0], 0, qn, qn + kn, q, qw.to(DEV), kw.to(DEV), True, None, None, 0, False, pos.to(DEV),
+                           seq.to(DEV), kc, vc, table.to(DEV), 128, 64, nh, nkv, hd, hdv, eps)
+        tol = 3e-6 if dtype == torch.float32 else 2 ** -7
+        assert rel_err(q, P.rms_norm(x[:, :qn], qw.double(), eps)) < tol
+        k = P.rms_norm(x[:, qn:qn + kn], kw.double(), eps).view(T, nkv, hd)
+        v = x[:, qn + kn:qn + kn + vn].reshape(T, nkv, hdv)
+        page = table[seq.long(), (pos.long() % 128) // 64].long()
+        assert rel_err(kc.cpu()[page, :, pos.long() % 64], k) < tol and rel_err(vc.cpu()[page, :, pos.long() % 64], v) < tol
+        used = torch.zeros(5, 64, dtype=torch.bool)
+        used[page, pos.long() % 64] = True
+        assert bool((kc.cpu().permute(0, 2, 1, 3)[~used] == 9.0).all()) and bool((vc.cpu().permute(0, 2, 1, 3)[~used] == 9.0).all())
+
+
 class _KV:
     def __init__(self, k, v, table, ring, window):
         self.k, self.v, self.table, self.ring, self.page, self.window, self.owner = k, v, table, ring, 64, window, True

@@ -336,6 +336,79 @@ qkv_place_rows_kernel(const TX* __restrict__ x, long long ldx, int n_parts, long
         for (int i = tid; i < g_width; i += blockDim.x) gate_out[t * g_width + i] = at(g_off + i);
 }
 
+// The same for rows that are [q | k | v] one behind the other, with the norms over all heads at once (or none), without rotation and
+// gate: the row stays in registers, four neighbouring columns a load (rows of up to 256 * 4 * NCH columns, sizes in fours), and one
+// round of the block makes both sums.
+template <typename TQ, typename TC, int NCH>
+__global__ void __launch_bounds__(256)
+qkv_place_whole_kernel(const float* __restrict__ x, long long ldx, int n_parts, long long part_stride, TQ* __restrict__ q_out,
+                       long long ldq, const float* __restrict__ qw, const float* __restrict__ kw, const int* __restrict__ tok_pos,
+                       const int* __restrict__ tok_seq, TC* __restrict__ kc, TC* __restrict__ vc, PagedKV c, PagedKV cv, int nh,
+                       float eps) {
+    __shared__ float red[2][8];
+    pdl_trigger();
+    const long long t = blockIdx.x;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int hd = c.head_dim, hdv = cv.head_dim, nkv = c.n_kv_heads;
+    const int qn = nh * hd, kn = nkv * hd, chunks = (qn + kn + nkv * hdv) >> 2;
+    const int pos = tok_pos[t], seq = tok_seq[t];
+    float4 w[NCH];
+#pragma unroll
+    for (int u = 0; u < NCH; ++u) {                         // the weights are there before the kernel ahead has ended
+        const int col = (tid + u * 256) * 4;
+        w[u] = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (qw && col < qn) w[u] = *reinterpret_cast<const float4*>(qw + col);
+        else if (kw && col >= qn && col < qn + kn) w[u] = *reinterpret_cast<const float4*>(kw + col - qn);
+    }
+    pdl_wait();
+    float4 v[NCH];
+#pragma unroll
+    for (int u = 0; u < NCH; ++u) v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int p = 0; p < n_parts; ++p) {
+        const float4* row = reinterpret_cast<const float4*>(x + p * part_stride + t * ldx);
+#pragma unroll
+        for (int u = 0; u < NCH; ++u) {
+            const int i = tid + u * 256;
+            if (i < chunks) {
+                const float4 a = row[i];
+                v[u].x += a.x; v[u].y += a.y; v[u].z += a.z; v[u].w += a.w;
+            }
+        }
+    }
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int u = 0; u < NCH; ++u) {
+        const int col = (tid + u * 256) * 4;
+        const float ss = (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
+        if (col < qn) sq += ss; else if (col < qn + kn) sk += ss;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
+    const float inv_q = qw ? inv_rms(sq, (float)qn, eps) : 1.f, inv_k = kw ? inv_rms(sk, (float)kn, eps) : 1.f;
+#pragma unroll
+    for (int u = 0; u < NCH; ++u) {
+        const int i = tid + u * 256, col = i * 4;
+        if (i >= chunks) break;
+        const float f = col < qn ? inv_q : col < qn + kn ? inv_k : 1.f;
+        const float e[4] = {v[u].x * f * w[u].x, v[u].y * f * w[u].y, v[u].z * f * w[u].z, v[u].w * f * w[u].w};
+        if (col < qn) {
+            store_vec<TQ, 4>(q_out + t * ldq + col, e);
+        } else if (col < qn + kn) {
+            const int k = col - qn;
+            store_vec<TC, 4>(kc + paged_offset(c, seq, pos, k / hd) + k % hd, e);
+        } else {
+            const int k = col - qn - kn;
+            store_vec<TC, 4>(vc + paged_offset(cv, seq, pos, k / hdv) + k % hdv, e);
+        }
+    }
+}
+
 UB_API int ub_qkv_place_rows(const void* x, int x_dtype, long long ldx, int n_parts, long long part_stride, int q_off, int k_off,
                              int v_off, void* q_out, int q_dtype, long long ldq, const float* qw, const float* kw, int norm_whole,
                              const float* cs, const float* sn, int rd, int interleaved, const int* tok_pos, const int* tok_seq,
@@ -350,6 +423,20 @@ UB_API int ub_qkv_place_rows(const void* x, int x_dtype, long long ldx, int n_pa
     PagedKV c{table, pages_per_seq, ring, page, nkv, hd};
     PagedKV cv{table, pages_per_seq, ring, page, nkv, hd_v};
     cudaError_t e;
+    const int cols = nh * hd + nkv * (hd + hd_v);
+    if (x_dtype == UB_F32 && (norm_whole || (!qw && !kw)) && !cs && !gate_out && q_off == 0 && k_off == nh * hd && v_off == (nh + nkv) * hd &&
+        hd % 4 == 0 && hd_v % 4 == 0 && ldx % 4 == 0 && part_stride % 4 == 0 && ldq % 4 == 0 && cols <= 256 * 4 * 16 &&
+        (((uintptr_t)x | (uintptr_t)q_out | (uintptr_t)qw | (uintptr_t)kw | (uintptr_t)kcache | (uintptr_t)vcache) & 15) == 0 &&
+        q_dtype == cache_dtype && (q_dtype == UB_F32 || q_dtype == UB_BF16)) {
+        const int nch = (cols / 4 + 255) / 256;
+#define GO2(TT, NCH) e = ub_launch_dependent(qkv_place_whole_kernel<TT, TT, NCH>, dim3(n_tokens), dim3(256), 0, st, (const float*)x, ldx, n_parts, \
+            part_stride, (TT*)q_out, ldq, qw, kw, tok_pos, tok_seq, (TT*)kcache, (TT*)vcache, c, cv, nh, eps)
+#define GO1(NCH) do { if (q_dtype == UB_F32) GO2(float, NCH); else GO2(__nv_bfloat16, NCH); } while (0)
+        if (nch <= 2) GO1(2); else if (nch <= 4) GO1(4); else if (nch <= 8) GO1(8); else GO1(16);
+#undef GO1
+#undef GO2
+        return (int)e;
+    }
 #define GO(TX, TQ, TC) do { \
         if (smem > 48 * 1024) cudaFuncSetAttribute(qkv_place_rows_kernel<TX, TQ, TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         e = ub_launch_dependent(qkv_place_rows_kernel<TX, TQ, TC>, dim3(n_tokens), dim3(256), smem, st, (const TX*)x, ldx, n_parts, \
