@@ -104,10 +104,18 @@ lin_gates_kernel(const float* __restrict__ p, LinShape s, const float* __restric
     if (t0 >= t1) return;
     float* ms = m_state + (long long)seq_slot[b] * s.H + h;
     float m = *ms;                                            // the maximum before this turn's first token
+    const float b_in = bi[h], b_forget = bf[h];
+    float zi = 0.f, zf = 0.f;                                 // a turn's sums are asked for while the turn before it is worked on
+    auto ask = [&](int t) {
+        if (t < t1) { zi = lin_at(p, s, t, s.x_off + h); zf = lin_at(p, s, t, s.y_off + h); }
+    };
+    ask(t0 + threadIdx.x);
     for (int base = t0; base < t1; base += GATE_WARPS * 32) {
         const int t = base + threadIdx.x;
+        const float yi = zi, yf = zf;
+        ask(t + GATE_WARPS * 32);
         float f1 = 0.f, i1 = -INFINITY;                       // past the end: the map that changes nothing
-        if (t < t1) log_gates(lin_at(p, s, t, s.x_off + h) + bi[h], lin_at(p, s, t, s.y_off + h) + bf[h], cap, i1, f1);
+        if (t < t1) log_gates(yi + b_in, yf + b_forget, cap, i1, f1);
         float f = f1, i = i1;                                 // the map of this warp's tokens up to and with this lane's
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {

@@ -96,6 +96,9 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
             if (gm[i / size] != INFINITY) ch[i] = -INFINITY;
         __syncwarp();
     }
+    const bool held = top <= 32;                          // choice k and its score stay with lane k
+    float mine = 0.f;
+    int mine_at = 0;
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
         int at = 0x7fffffff;
@@ -109,13 +112,27 @@ __device__ __forceinline__ void route_token(const float* __restrict__ zr, int n_
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (at == 0x7fffffff) at = 0;                     // (every score was taken or not a number: a row of NaN)
+        if (held && lane == k) { mine = sc[at]; mine_at = at; }
         if (lane == 0) {
-            idx_t[k] = at;
-            wts_t[k] = sc[at];
+            if (!held) { idx_t[k] = at; wts_t[k] = sc[at]; }
             ch[at] = NAN;                                 // taken: NaN is passed over, while -inf may still be chosen
             if (at < n_experts) atomicAdd(&counts[at], 1);
         }
         __syncwarp();
+    }
+    if (held) {
+        const bool has = lane < top;
+        if (mode & 8) {
+            const float top_z = warp_max(has ? mine : -INFINITY);
+            mine = has ? expf(mine - top_z) : 0.f;
+            mine = mine / warp_sum(mine) * wscale;
+        } else if (mode & 4) {
+            mine *= wscale / (warp_sum(has ? mine : 0.f) + 1e-20f);
+        } else {
+            mine *= wscale;
+        }
+        if (has) { idx_t[lane] = mine_at; wts_t[lane] = mine; }
+        return;
     }
     if (lane == 0 && (mode & 8)) {
         float top_z = -INFINITY, sum = 0.f;
