@@ -492,6 +492,7 @@ ONE_LAYER = {
     "parallel_equal_sizes": _model([_layer(_par((4, 4, 64, 64, 0.12, 64), (4, 32, 32, 16.0, 32)))], width=64),
     "parallel_window_of_one": _model([_layer(_par((2, 1, 48, 32, 0.3, 1), (1, 64, 96, 2.0, 7)))], eps=1e-3),
     "parallel_no_fours": _model([_layer(_par((3, 1, 10, 14, 0.3, 30), (3, 11, 13, 1.0, 5)))], width=50),
+    "parallel_large_heads": _model([_layer(_par((2, 1, 160, 320, 0.08, 45), (1, 128, 288, 4.0, 24)))], width=72),
     "routed": _model([_layer(_SMALL, _moe(10, 3, 24))], width=72),
     "routed_all_chosen": _model([_layer(_SMALL, _moe(3, 3, 128))], width=48),
     "routed_no_eights": _model([_layer(_SMALL, _moe(6, 1, 21))], width=50),

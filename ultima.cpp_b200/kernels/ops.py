@@ -14,6 +14,7 @@ from . import build
 F32, BF16 = 0, 1
 EPI_STORE, EPI_ADD, EPI_SWIGLU, EPI_SWIGLU_IL = 0, 1, 2, 3
 MAX_HEAD_DIM = 256          # the largest head size the attention and q/k preparation kernels take
+MAX_KEY_ROW, MAX_VALUE_ROW = 1024, 512       # the largest key and value rows of the any-shape attention kernel
 
 
 class KernelError(RuntimeError):

@@ -211,9 +211,11 @@ class Attention(Mixer):
                 and self.block is None and not self.head_gate and self.own_kv)
 
     def bind(self, tensors, rt):
-        if (self.hd % 2 and not self.general) or self.hd > ops.MAX_HEAD_DIM or self.hdv > ops.MAX_HEAD_DIM:
-            raise ValueError(f"attention: head size {self.hd} is not one the kernels take (even, at most "
-                             f"{ops.MAX_HEAD_DIM})")
+        # the row-wise placement and the any-shape attention kernel take larger heads than the others
+        most = (ops.MAX_KEY_ROW, ops.MAX_VALUE_ROW) if self.place_rows else (ops.MAX_HEAD_DIM, ops.MAX_HEAD_DIM)
+        if (self.hd % 2 and not self.general) or self.hd > most[0] or self.hdv > most[1]:
+            raise ValueError(f"attention: head size {self.hd} is not one the kernels take (even, at most {most[0]}; values, here "
+                             f"{self.hdv}, at most {most[1]})")
         ws = [tensors["q_proj.weight"]]
         if self.own_kv:
             ws.append(tensors["k_proj.weight"])
